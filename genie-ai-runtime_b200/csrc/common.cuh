@@ -184,6 +184,7 @@ inline cudaError_t launch_k(void (*kern)(KArgs...), dim3 grid, dim3 block, size_
     return cudaLaunchKernelEx(&cfg, kern, KArgs(args)...);
 }
 
+const void* resolve_weight(const void* W);   // device pointer of a weight tensor (registered host ranges are mapped)
 bool pdl_enabled();          // process-wide switch (default on)
 void count_launch(int n = 1);  // launch counter for the benchmark's gpu_launches claim
 

@@ -1,0 +1,49 @@
+// decoder.cuh — the decoder session: one request stream with the position and the token in device memory, so that one
+// captured CUDA graph serves every step.  The session (decoder.cu) owns the stream state, the greedy token, the graph and
+// the cutting of prompts into chunks; what a step or a chunk computes is the model family's, behind the virtual
+// functions: decoder_kquant.cu (GGUF K-quant Llama / Qwen3 layers, also tensor-parallel) and decoder_layers.cu (models
+// described layer by layer).
+#pragma once
+#include "../../include/jllm_b200.h"
+#include "common.cuh"
+
+#define DCHK(call) do { const int rc__ = (call); if (rc__) return rc__; } while (0)
+
+struct jllm_b200_decoder {
+    // ── session state ──
+    int vocab = 0, max_context = 0;      // vocab: rows of this rank's logits
+    int vocab_full = 0;
+    bool use_graph = false;
+    bool batched_prefill = false;        // generate() runs the prompt through the chunk path
+    float* logits = nullptr;             // [vocab] of the last step
+    int* state = nullptr;                // [0..3] position, token, tokens recorded; [32..] argmax scratch; [200..] barrier words
+    int* out_tokens = nullptr; int out_cap = 0;
+    int* prompt_dev = nullptr; int prompt_cap = 0;
+    cudaGraphExec_t graph_exec = nullptr; int graph_splits = 0;
+    int host_pos = 0;                    // host mirror of the device-side position (next step's position)
+    cudaStream_t own_stream = nullptr;   // used when the caller passes the legacy default stream, which cannot be captured
+    int kernels_per_step = 0;
+    int pf_chunk = 2048, pf_cap = 0;     // prompt tokens per chunk; tokens the chunk buffers hold
+    int* pf_tokens = nullptr;
+    float* row_logits = nullptr; size_t row_logits_cap = 0;     // logits of the positions a feed asks for
+    void* session_slab = nullptr;
+
+    virtual ~jllm_b200_decoder() = default;
+    // ── the model family ──
+    virtual int enqueue_step(int n_splits, cudaStream_t st) = 0;              // token and position from `state`; leaves logits, then launch_argmax_advance (or its own)
+    virtual int reserve_chunk(int tokens) = 0;                                // buffers of a chunk (grown on first use)
+    virtual int enqueue_chunk(const int* dev_tokens, int n, int start, cudaStream_t st) = 0;
+    virtual int enqueue_rows(const int* host_rows, int n, float* out, cudaStream_t st) = 0;   // final norm + logits [n][vocab] of rows of the chunk just enqueued
+    virtual int attn_splits(int seq_len) const = 0;                           // KV slices of a step at this length (a graph is captured per value)
+    virtual bool has_chunks() const { return true; }
+    virtual void clear_cache() = 0;
+    virtual const void* buffer(int which) = 0;
+
+    int  session_alloc();                                                     // after vocab / max_context are set
+    void session_free();
+};
+
+namespace jb {
+// greedy token of fp32 logits [vocab]; records it and advances the step state
+int launch_argmax_advance(jllm_b200_decoder* d, cudaStream_t st);
+}

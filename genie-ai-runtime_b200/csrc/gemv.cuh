@@ -44,7 +44,6 @@ struct GemvTpPush { unsigned char* peer[8]; int world; int buf_off; int row_off;
 void gemv_set_tp_hooks(const GemvTpWait* wait, const GemvTpPush* push);
 
 // dispatch helpers shared with the decoder's chained launches (csrc/api.cu)
-const void* resolve_weight(const void* W);          // device pointer of a weight tensor (registered host ranges are mapped)
 bool triple_dp4a(int t0, int t1, int t2);            // type mixes the reference runs on its q8_1 + dp4a path
 
 int launch_gemv(const GemvArgs& a, cudaStream_t st);

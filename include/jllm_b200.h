@@ -257,6 +257,11 @@ int    jllm_b200_decoder_generate(jllm_b200_decoder* d, const int* host_prompt, 
  * not available in a tensor-parallel session. */
 int    jllm_b200_decoder_prefill(jllm_b200_decoder* d, const int* host_tokens, int n_tokens, int start_pos, void* stream);
 int    jllm_b200_decoder_set_prefill_chunk(jllm_b200_decoder* d, int tokens);
+/* Feeds n_tokens >= 1 host token ids at positions start_pos .. and returns the logits at the wanted places among them
+ * (`want`: rising indices into host_tokens): host_logits receives [n_want][vocab_size] floats.  One token runs the decode
+ * step, more run the chunk path; nothing is sampled.  The cache must hold positions 0 .. start_pos - 1.  Waits for the result. */
+int    jllm_b200_decoder_feed(jllm_b200_decoder* d, const int* host_tokens, int n_tokens, int start_pos, const int* want, int n_want,
+                              float* host_logits, void* stream);
 /* One step with the host boundary inside: host_pos_token = {position, token} (pinned host memory recommended) is copied
  * to the device, the step runs, the greedy token is copied to *host_next and the call returns once it has arrived. */
 int    jllm_b200_decoder_step_sync(jllm_b200_decoder* d, const int* host_pos_token, int* host_next, void* stream);
