@@ -1,11 +1,11 @@
 // attention.cuh — host-side call block of the attention kernels.
 #pragma once
-#include "common.cuh"
+#include "layernorm.cuh"
 
 namespace jb {
 
 struct AttnCall {
-    __half* out = nullptr; const __half* q = nullptr;
+    void* out = nullptr; const void* q = nullptr;      // fp16, or the cache's type when that is BF16 / FP32
     const void* k = nullptr; const void* v = nullptr; const float* ks = nullptr; const float* vs = nullptr;
     // ragged batch: device arrays of per-sequence pointers / lengths (batch entries)
     const void* const* k_list = nullptr; const void* const* v_list = nullptr;
@@ -18,18 +18,25 @@ struct AttnCall {
     const int* d_pos = nullptr;       // device position: seq_len = *d_pos + 1
     float scale = 1.f; int kv_int8 = 0, window = 0, n_splits = 0;
     int causal_start = -1;            // >= 0: prefill, `batch` = number of query tokens
+    // BF16 / FP32 caches (kv_kind overrides kv_int8): own value head size, row strides of q and out, softmax sink per query
+    // head, query temperature 1 + qt_coef * ln(floor((p + 1) / qt_every) + 1) at position p
+    int kv_kind = -1, vhd = 0, ldq = 0, ldo = 0;
+    const float* sink = nullptr;
+    float qt_coef = 0.f; double qt_every = 0.0;
+    int kind() const { return kv_kind >= 0 ? kv_kind : kv_int8 ? EK_INT8 : EK_F16; }
 };
 
 int    attn_splits_for(int seq_len);
 float* splitk_buffer(size_t floats, bool may_alloc);
 int    launch_attention_general(const AttnCall& c, cudaStream_t st);
 int    launch_attention(const AttnCall& c, cudaStream_t st);      // picks the fast path when it applies
-int    launch_attn_reduce(__half* out, const float* part, int n_heads, int hd, int n_splits, int batch, cudaStream_t st);
-unsigned int* attn_tickets();                                     // 65536 zeroed words per device (slice counters of the TMA kernel)
 bool   attention_tma_applies(const AttnCall& c);                  // INT8 KV, head_dim 128, GQA 1/2/4, no window, cache extent known
 int    launch_attention_tma(const AttnCall& c, cudaStream_t st);
 bool   attn_tma_encode(void* map_out128, const void* cache_base, int rows, int n_kv);
 bool   attention_prefill_fast_applies(const AttnCall& c);          // causal prefill (causal_start >= 0), INT8 KV, head_dim 128, GQA 1/2/4
 int    launch_attention_prefill_fast(const AttnCall& c, cudaStream_t st);
+bool   attention_bf16_applies(const AttnCall& c);                  // BF16 cache, head sizes multiples of 8 up to 256: decode and causal prefill
+int    launch_attention_bf16(const AttnCall& c, cudaStream_t st);
+int    attn_bf16_splits(int seq_len, int n_heads, int n_kv);       // KV slices of a decode call at this length
 
 }  // namespace jb

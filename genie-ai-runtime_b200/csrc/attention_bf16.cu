@@ -1,0 +1,418 @@
+// attention_bf16.cu — attention over a BF16 KV cache on tensor cores (mma.sync m16n8k16, fp32 accumulate): causal prefill
+// with query tiling and split-KV decode, for any head sizes that are multiples of 8 up to 256 (keys and values may differ)
+// and any GQA ratio, with an optional softmax sink and query temperature.
+//
+// Both kernels pack (token, query head of the group) pairs as the 16 rows of an MMA tile, so the query heads that share a
+// KV head share every K / V byte.  Scores, softmax weights and their sums are fp32; the weights are rounded to bf16 as the
+// operand of the second product only.  K / V rows are staged by 16-byte cp.async copies into rows of D elements whose
+// 16-byte chunks are XOR-swizzled by the row (conflict-free ldmatrix); D = 64, 128 or 256 is the larger head size rounded
+// up, and k-steps / output tiles beyond the real sizes are skipped.
+#include "attention.cuh"
+#include "attention_general.cuh"
+
+namespace jb {
+
+struct FaArgs {
+    __nv_bfloat16* out; const __nv_bfloat16* q; const __nv_bfloat16* k; const __nv_bfloat16* v;
+    int n_heads, n_kv, R;            // R = query heads per KV head
+    int dim, vdim, ldq, ldo, ldk, ldv;
+    int n_tokens, start;             // prefill
+    int seq_len; const int* d_pos;   // decode: keys = *d_pos + 1 when d_pos is given
+    int n_splits, row_blocks;        // decode: KV slices; blocks of 16 query heads per KV head
+    float scale; const float* sink; float qt_coef; double qt_every;
+    float* part; unsigned int* tickets;
+};
+
+constexpr float FA_LOG2E = 1.4426950408889634f;
+
+__device__ __forceinline__ void fa_cp16(uint32_t dst, const void* src, bool in) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(in ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void fa_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N> __device__ __forceinline__ void fa_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+__device__ __forceinline__ void fa_ldsm(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void fa_ldsm_t(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void fa_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ uint32_t fa_pack(float lo, float hi) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(lo, hi);
+    return *reinterpret_cast<const uint32_t*>(&h);
+}
+// byte offset of 16-byte chunk c of row r in a tile of D-element rows
+template <int D> __device__ __forceinline__ uint32_t fa_off(int r, int c) { return (uint32_t)(r * D * 2 + ((c ^ (r & 7)) << 4)); }
+
+// One 16-row step over NK keys (a multiple of 16) whose K / V tiles sit in shared memory: S = Q K^T, online softmax in base
+// 2, O += P V.  qf(ks) gives the A fragment of k-step ks.  live(row_half, key) masks; fsc[2] = score factors of the two rows.
+template <int D, int NK, class QF, class Live>
+__device__ __forceinline__ void fa_step(float (&o)[D / 8][4], float (&m)[2], float (&l)[2], const float (&fsc)[2], uint32_t ks_addr, uint32_t vs_addr,
+                                        int dim, int vdim, bool masked, QF qf, Live live) {
+    const int lane = threadIdx.x & 31, lr = lane & 7, lm = lane >> 3;
+    float s[NK / 8][4];
+    #pragma unroll
+    for (int i = 0; i < NK / 8; ++i) { s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f; }
+    #pragma unroll
+    for (int ks = 0; ks < D / 16; ++ks) {
+        if (ks * 16 < dim) {
+            uint32_t a[4];
+            qf(ks, a);
+            #pragma unroll
+            for (int nt = 0; nt < NK / 16; ++nt) {           // matrices: keys 0-7 | 8-15 of the pair, k halves
+                uint32_t b[4];
+                fa_ldsm(b, ks_addr + fa_off<D>(nt * 16 + (lm >> 1) * 8 + lr, ks * 2 + (lm & 1)));
+                fa_mma(s[2 * nt], a, b[0], b[1]);
+                fa_mma(s[2 * nt + 1], a, b[2], b[3]);
+            }
+        }
+    }
+    float mx[2] = {-INFINITY, -INFINITY};
+    #pragma unroll
+    for (int i = 0; i < NK / 8; ++i)
+        #pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            float v = s[i][e] * fsc[e >> 1];
+            if (masked && !live(e >> 1, i * 8 + (lane & 3) * 2 + (e & 1))) v = -INFINITY;
+            s[i][e] = v;
+            mx[e >> 1] = fmaxf(mx[e >> 1], v);
+        }
+    float corr[2], sum[2] = {0.f, 0.f};
+    #pragma unroll
+    for (int h = 0; h < 2; ++h) {
+        mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xFFFFFFFFu, mx[h], 1));
+        mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xFFFFFFFFu, mx[h], 2));
+        const float mn = fmaxf(m[h], mx[h]);
+        corr[h] = mn == -INFINITY ? 1.f : exp2f(m[h] - mn);         // no key seen yet: nothing to rescale
+        m[h] = mn;
+    }
+    #pragma unroll
+    for (int i = 0; i < NK / 8; ++i)
+        #pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const float mm = m[e >> 1];
+            const float p = mm == -INFINITY ? 0.f : exp2f(s[i][e] - mm);
+            s[i][e] = p;
+            sum[e >> 1] += p;
+        }
+    #pragma unroll
+    for (int h = 0; h < 2; ++h) l[h] = l[h] * corr[h] + sum[h];     // lane-private part of the row sum; reduced at the end
+    #pragma unroll
+    for (int dt = 0; dt < D / 8; ++dt) { o[dt][0] *= corr[0]; o[dt][1] *= corr[0]; o[dt][2] *= corr[1]; o[dt][3] *= corr[1]; }
+    #pragma unroll
+    for (int kk = 0; kk < NK / 16; ++kk) {
+        const uint32_t a[4] = {fa_pack(s[2 * kk][0], s[2 * kk][1]), fa_pack(s[2 * kk][2], s[2 * kk][3]),
+                               fa_pack(s[2 * kk + 1][0], s[2 * kk + 1][1]), fa_pack(s[2 * kk + 1][2], s[2 * kk + 1][3])};
+        #pragma unroll
+        for (int dt = 0; dt < D / 16; ++dt) {
+            if (dt * 16 < vdim) {                            // transposed matrices: keys 0-7 | 8-15, then the next 8 dims
+                uint32_t b[4];
+                fa_ldsm_t(b, vs_addr + fa_off<D>(kk * 16 + (lm & 1) * 8 + lr, dt * 2 + (lm >> 1)));
+                fa_mma(o[2 * dt], a, b[0], b[1]);
+                fa_mma(o[2 * dt + 1], a, b[2], b[3]);
+            }
+        }
+    }
+}
+
+// rows [row0, row0 + n) of a cache matrix into a swizzled tile; chunks up to the 16-element round-up of `width`, zero beyond
+// the real width and beyond row `end`
+template <int D>
+__device__ __forceinline__ void fa_load_rows(uint32_t tile, const __nv_bfloat16* base, int ld, int width, int row0, int n, int end, int tid, int threads) {
+    const int ch = ((width + 15) >> 4) * 2, real = width >> 3;
+    for (int i = tid; i < n * ch; i += threads) {
+        const int r = i / ch, c = i - r * ch;
+        const bool in = row0 + r < end && c < real;
+        fa_cp16(tile + fa_off<D>(r, c), in ? base + (size_t)(row0 + r) * ld + c * 8 : base, in);
+    }
+}
+
+// ── causal prefill: 64 rows (4 warps x 16) against tiles of 64 keys ──
+constexpr int FP_ROWS = 64, FP_KEYS = 64, FP_THREADS = 128;
+template <int D> constexpr bool fp_q_in_regs() { return D <= 128; }
+// two stages of K and V; the query tile shares the second K stage when its fragments live in registers
+template <int D> constexpr int fp_smem() { return (4 + (fp_q_in_regs<D>() ? 0 : 1)) * FP_KEYS * D * 2; }
+
+template <int D>
+__global__ void __launch_bounds__(FP_THREADS) attn_bf16_prefill_kernel(const FaArgs a) {
+    pdl_wait();
+    extern __shared__ __align__(128) unsigned char fp_sm[];
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int g = blockIdx.y, tile = gridDim.x - 1 - blockIdx.x;        // longest tiles first
+    const int total = a.n_tokens * a.R, row0 = tile * FP_ROWS;
+    constexpr uint32_t TB = FP_KEYS * D * 2;
+    const uint32_t sm = smem_u32(fp_sm), qst = fp_q_in_regs<D>() ? sm + TB : sm + 4 * TB;
+    const int last_tok = (min(row0 + FP_ROWS, total) - 1) / a.R, n_keys = a.start + last_tok + 1;
+    const __nv_bfloat16* kb = a.k + (size_t)g * a.dim;
+    const __nv_bfloat16* vb = a.v + (size_t)g * a.vdim;
+    {   // query rows: (token, head of the group)
+        const int ch = ((a.dim + 15) >> 4) * 2, real = a.dim >> 3;
+        for (int i = tid; i < FP_ROWS * ch; i += FP_THREADS) {
+            const int r = i / ch, c = i - r * ch, fr = row0 + r;
+            const bool in = fr < total && c < real;
+            const int t = fr / a.R, h = g * a.R + fr - t * a.R;
+            fa_cp16(qst + fa_off<D>(r, c), in ? a.q + (size_t)t * a.ldq + (size_t)h * a.dim + c * 8 : a.q, in);
+        }
+        fa_commit();
+    }
+    fa_load_rows<D>(sm, kb, a.ldk, a.dim, 0, FP_KEYS, n_keys, tid, FP_THREADS);
+    fa_load_rows<D>(sm + 2 * TB, vb, a.ldv, a.vdim, 0, FP_KEYS, n_keys, tid, FP_THREADS);
+    fa_commit();
+    uint32_t qreg[fp_q_in_regs<D>() ? D / 16 : 1][4];
+    const uint32_t q_lane = (uint32_t)(warp * 16 + (lane & 15));
+    if (fp_q_in_regs<D>()) {
+        fa_wait<1>();
+        __syncthreads();
+        #pragma unroll
+        for (int ks = 0; ks < D / 16; ++ks) if (ks * 16 < a.dim) fa_ldsm(qreg[fp_q_in_regs<D>() ? ks : 0], qst + fa_off<D>((int)q_lane, ks * 2 + (lane >> 4)));
+        __syncthreads();                                   // the second K stage is free for keys
+    }
+    auto qf = [&](int ks, uint32_t (&f)[4]) {
+        if constexpr (fp_q_in_regs<D>()) { f[0] = qreg[ks][0]; f[1] = qreg[ks][1]; f[2] = qreg[ks][2]; f[3] = qreg[ks][3]; }
+        else fa_ldsm(f, qst + fa_off<D>((int)q_lane, ks * 2 + (lane >> 4)));
+    };
+    int pos[2];
+    float fsc[2], m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f}, o[D / 8][4];
+    #pragma unroll
+    for (int h = 0; h < 2; ++h) {
+        const int fr = min(row0 + warp * 16 + (lane >> 2) + 8 * h, total - 1);
+        pos[h] = a.start + fr / a.R;
+        fsc[h] = a.scale * q_temp_factor(pos[h], a.qt_coef, a.qt_every) * FA_LOG2E;
+    }
+    #pragma unroll
+    for (int i = 0; i < D / 8; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
+    const int warp_first = a.start + min(row0 + warp * 16, total - 1) / a.R;            // least position among the warp's rows
+    const int warp_last = a.start + min(row0 + warp * 16 + 15, total - 1) / a.R;
+    const int tiles = (n_keys + FP_KEYS - 1) / FP_KEYS;
+    for (int t = 0; t < tiles; ++t) {
+        const uint32_t b = t & 1;
+        if (t + 1 < tiles) {
+            fa_load_rows<D>(sm + (b ^ 1) * TB, kb, a.ldk, a.dim, (t + 1) * FP_KEYS, FP_KEYS, n_keys, tid, FP_THREADS);
+            fa_load_rows<D>(sm + (2 + (b ^ 1)) * TB, vb, a.ldv, a.vdim, (t + 1) * FP_KEYS, FP_KEYS, n_keys, tid, FP_THREADS);
+        }
+        fa_commit();
+        fa_wait<1>();
+        __syncthreads();
+        const int k0 = t * FP_KEYS;
+        if (k0 <= warp_last)
+            fa_step<D, FP_KEYS>(o, m, l, fsc, sm + b * TB, sm + (2 + b) * TB, a.dim, a.vdim, k0 + FP_KEYS - 1 > warp_first, qf, [&](int h, int key) { return k0 + key <= pos[h]; });
+        __syncthreads();
+    }
+    #pragma unroll
+    for (int h = 0; h < 2; ++h) {
+        float L = l[h];
+        L += __shfl_xor_sync(0xFFFFFFFFu, L, 1);
+        L += __shfl_xor_sync(0xFFFFFFFFu, L, 2);
+        const int fr = row0 + warp * 16 + (lane >> 2) + 8 * h;
+        if (fr >= total) continue;
+        const int t = fr / a.R, head = g * a.R + fr - t * a.R;
+        const float inv = sink_norm(m[h] / FA_LOG2E, L, a.sink ? a.sink + head : nullptr);
+        __nv_bfloat16* out = a.out + (size_t)t * a.ldo + (size_t)head * a.vdim;
+        #pragma unroll
+        for (int dt = 0; dt < D / 8; ++dt) {
+            const int d = dt * 8 + (lane & 3) * 2;
+            if (d < a.vdim) *reinterpret_cast<uint32_t*>(out + d) = fa_pack(o[dt][2 * h] * inv, o[dt][2 * h + 1] * inv);
+        }
+    }
+}
+
+// ── decode: one CTA per (KV head, block of 16 query heads, KV slice); every warp runs its own ring of 16-key tiles ──
+constexpr int FD_WARPS = 4, FD_THREADS = FD_WARPS * 32, FD_KEYS = 16;
+template <int D> constexpr int fd_stages() { return D == 256 ? 2 : D == 128 ? 3 : 6; }
+template <int D> constexpr int fd_smem() {
+    return FD_WARPS * fd_stages<D>() * 2 * FD_KEYS * D * 2 > FD_WARPS * 16 * (D + 2) * 4 ? FD_WARPS * fd_stages<D>() * 2 * FD_KEYS * D * 2 : FD_WARPS * 16 * (D + 2) * 4;
+}
+
+template <int D>
+__global__ void __launch_bounds__(FD_THREADS) attn_bf16_decode_kernel(const FaArgs a) {
+    pdl_wait();
+    extern __shared__ __align__(128) unsigned char fd_sm[];
+    __shared__ int last;
+    constexpr int ST = fd_stages<D>();
+    constexpr uint32_t TB = FD_KEYS * D * 2;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int g = blockIdx.x / a.row_blocks, rb = blockIdx.x - g * a.row_blocks, split = blockIdx.y;
+    const int h0 = g * a.R + rb * 16, n_rows = min(16, a.R - rb * 16);
+    const int seq = a.d_pos ? *a.d_pos + 1 : a.seq_len;
+    const int per = (((seq + a.n_splits - 1) / a.n_splits) + FD_KEYS - 1) / FD_KEYS * FD_KEYS;
+    const int k_lo = min(split * per, seq), k_hi = min(k_lo + per, seq);
+    const __nv_bfloat16* kb = a.k + (size_t)g * a.dim;
+    const __nv_bfloat16* vb = a.v + (size_t)g * a.vdim;
+    const uint32_t ring = smem_u32(fd_sm) + (uint32_t)warp * ST * 2 * TB;
+    // query fragments straight from global memory: row = head, columns 2 (lane & 3) .. of each k half
+    uint32_t qreg[D / 16][4];
+    #pragma unroll
+    for (int ks = 0; ks < D / 16; ++ks)
+        #pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int r = (lane >> 2) + 8 * (i & 1), d = ks * 16 + (i >> 1) * 8 + (lane & 3) * 2;
+            qreg[ks][i] = r < n_rows && d < a.dim ? *reinterpret_cast<const uint32_t*>(a.q + (size_t)(h0 + r) * a.dim + d) : 0u;
+        }
+    const float f = a.scale * q_temp_factor(seq - 1, a.qt_coef, a.qt_every) * FA_LOG2E, fsc[2] = {f, f};
+    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f}, o[D / 8][4];
+    #pragma unroll
+    for (int i = 0; i < D / 8; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
+    const int tiles = (k_hi - k_lo + FD_KEYS - 1) / FD_KEYS, mine = tiles > warp ? (tiles - warp + FD_WARPS - 1) / FD_WARPS : 0;
+    auto fetch = [&](int i) {
+        const int k0 = k_lo + (warp + i * FD_WARPS) * FD_KEYS;
+        const uint32_t st = ring + (uint32_t)(i % ST) * 2 * TB;
+        fa_load_rows<D>(st, kb, a.ldk, a.dim, k0, FD_KEYS, k_hi, lane, 32);
+        fa_load_rows<D>(st + TB, vb, a.ldv, a.vdim, k0, FD_KEYS, k_hi, lane, 32);
+    };
+    #pragma unroll
+    for (int i = 0; i < ST - 1; ++i) { if (i < mine) fetch(i); fa_commit(); }
+    for (int i = 0; i < mine; ++i) {
+        fa_wait<ST - 2>();
+        __syncwarp();
+        const int k0 = k_lo + (warp + i * FD_WARPS) * FD_KEYS;
+        const uint32_t st = ring + (uint32_t)(i % ST) * 2 * TB;
+        fa_step<D, FD_KEYS>(o, m, l, fsc, st, st + TB, a.dim, a.vdim, k0 + FD_KEYS > k_hi,
+                            [&](int ks, uint32_t (&fr)[4]) { for (int e = 0; e < 4; ++e) fr[e] = qreg[ks][e]; }, [&](int, int key) { return k0 + key < k_hi; });
+        __syncwarp();
+        if (i + ST - 1 < mine) fetch(i + ST - 1);
+        fa_commit();
+    }
+    fa_wait<0>();
+    __syncthreads();                                       // the ring becomes the merge buffer
+    float* sm_m = reinterpret_cast<float*>(fd_sm);         // [warp][16]
+    float* sm_l = sm_m + FD_WARPS * 16;
+    float* sm_o = sm_l + FD_WARPS * 16;                    // [warp][16][D]
+    #pragma unroll
+    for (int h = 0; h < 2; ++h) {
+        float L = l[h];
+        L += __shfl_xor_sync(0xFFFFFFFFu, L, 1);
+        L += __shfl_xor_sync(0xFFFFFFFFu, L, 2);
+        const int r = (lane >> 2) + 8 * h;
+        if ((lane & 3) == 0) { sm_m[warp * 16 + r] = m[h]; sm_l[warp * 16 + r] = L; }
+        if (r < n_rows) {
+            #pragma unroll
+            for (int dt = 0; dt < D / 8; ++dt) {
+                const int d = dt * 8 + (lane & 3) * 2;
+                *reinterpret_cast<float2*>(sm_o + (size_t)(warp * 16 + r) * D + d) = make_float2(o[dt][2 * h], o[dt][2 * h + 1]);
+            }
+        }
+    }
+    __syncthreads();
+    const int rec = a.vdim + 2;
+    for (int r = warp; r < n_rows; r += FD_WARPS) {
+        float M = -INFINITY, L = 0.f, e[FD_WARPS];
+        #pragma unroll
+        for (int w = 0; w < FD_WARPS; ++w) M = fmaxf(M, sm_m[w * 16 + r]);
+        #pragma unroll
+        for (int w = 0; w < FD_WARPS; ++w) { e[w] = M == -INFINITY ? 0.f : exp2f(sm_m[w * 16 + r] - M); L += sm_l[w * 16 + r] * e[w]; }
+        const int head = h0 + r;
+        if (a.n_splits == 1) {
+            const float inv = sink_norm(M / FA_LOG2E, L, a.sink ? a.sink + head : nullptr);
+            for (int d = lane; d < a.vdim; d += 32) {
+                float acc = 0.f;
+                #pragma unroll
+                for (int w = 0; w < FD_WARPS; ++w) acc += sm_o[(size_t)(w * 16 + r) * D + d] * e[w];
+                a.out[(size_t)head * a.vdim + d] = __float2bfloat16_rn(acc * inv);
+            }
+        } else {
+            float* pb = a.part + ((size_t)head * a.n_splits + split) * rec;
+            for (int d = lane; d < a.vdim; d += 32) {
+                float acc = 0.f;
+                #pragma unroll
+                for (int w = 0; w < FD_WARPS; ++w) acc += sm_o[(size_t)(w * 16 + r) * D + d] * e[w];
+                pb[2 + d] = acc;
+            }
+            if (lane == 0) { pb[0] = M; pb[1] = L; }
+        }
+    }
+    if (a.n_splits == 1) return;
+    // the last CTA of this block of heads to finish merges the slices (a ticket, no waiting) and leaves the ticket at zero
+    __threadfence();
+    __syncthreads();
+    if (tid == 0) last = atomicAdd(&a.tickets[blockIdx.x], 1u) == (unsigned)a.n_splits - 1;
+    __syncthreads();
+    if (!last) return;
+    __threadfence();
+    if (tid == 0) a.tickets[blockIdx.x] = 0u;
+    for (int r = warp; r < n_rows; r += FD_WARPS) {
+        const int head = h0 + r;
+        const float* pb = a.part + (size_t)head * a.n_splits * rec;
+        float M = -INFINITY, L = 0.f;
+        for (int s = lane; s < a.n_splits; s += 32) M = fmaxf(M, __ldcg(pb + (size_t)s * rec));
+        M = warp_max(M);
+        for (int s = lane; s < a.n_splits; s += 32) { const float ms = __ldcg(pb + (size_t)s * rec); L += ms == -INFINITY ? 0.f : __ldcg(pb + (size_t)s * rec + 1) * exp2f(ms - M); }
+        L = warp_sum(L);
+        const float inv = sink_norm(M / FA_LOG2E, L, a.sink ? a.sink + head : nullptr);
+        float acc[D / 32];
+        #pragma unroll
+        for (int i = 0; i < D / 32; ++i) acc[i] = 0.f;
+        #pragma unroll 4
+        for (int s = 0; s < a.n_splits; ++s) {
+            const float ms = __ldcg(pb + (size_t)s * rec), e = ms == -INFINITY ? 0.f : exp2f(ms - M);
+            #pragma unroll
+            for (int i = 0; i < D / 32; ++i) { const int d = lane + 32 * i; if (d < a.vdim) acc[i] += __ldcg(pb + (size_t)s * rec + 2 + d) * e; }
+        }
+        #pragma unroll
+        for (int i = 0; i < D / 32; ++i) { const int d = lane + 32 * i; if (d < a.vdim) a.out[(size_t)head * a.vdim + d] = __float2bfloat16_rn(acc[i] * inv); }
+    }
+}
+
+// ── host side ──
+bool attention_bf16_applies(const AttnCall& c) {
+    const int vd = c.vhd > 0 ? c.vhd : c.hd;
+    return c.kind() == EK_BF16 && c.hd > 0 && c.hd <= 256 && vd > 0 && vd <= 256 && c.hd % 8 == 0 && vd % 8 == 0 && c.chd == c.hd && c.window == 0 && !c.k_list &&
+           c.k && c.v && !((uintptr_t)c.k & 15) && !((uintptr_t)c.v & 15) && !((uintptr_t)c.q & 15) && !((uintptr_t)c.out & 3) && c.ldq % 8 == 0 && c.ldo % 2 == 0 &&
+           c.n_kv > 0 && c.n_heads % c.n_kv == 0;
+}
+// Slices double with the length (a session captures one graph per value): at least 128 keys each, and no more CTAs than two per SM.
+int attn_bf16_splits(int seq_len, int n_heads, int n_kv) {
+    const int blocks = n_kv * ((n_heads / n_kv + 15) / 16);
+    int n = 1;
+    while (n < 64 && seq_len >= 256 * n && 2 * n * blocks <= 296) n *= 2;
+    return n;
+}
+
+template <int D>
+static int fa_launch(const FaArgs& a, bool prefill, cudaStream_t st) {
+    static bool attr = false;
+    if (!attr) {
+        JB_CUDA(cudaFuncSetAttribute(attn_bf16_prefill_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, fp_smem<D>()));
+        JB_CUDA(cudaFuncSetAttribute(attn_bf16_decode_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, fd_smem<D>()));
+        attr = true;
+    }
+    if (prefill) {
+        const long long rows = (long long)a.n_tokens * a.R;
+        JB_CUDA(launch_k(attn_bf16_prefill_kernel<D>, dim3((unsigned)((rows + FP_ROWS - 1) / FP_ROWS), a.n_kv), dim3(FP_THREADS), fp_smem<D>(), st, pdl_enabled(), a));
+    } else {
+        JB_CUDA(launch_k(attn_bf16_decode_kernel<D>, dim3(a.n_kv * a.row_blocks, a.n_splits), dim3(FD_THREADS), fd_smem<D>(), st, pdl_enabled(), a));
+    }
+    count_launch();
+    return JB_OK;
+}
+
+int launch_attention_bf16(const AttnCall& c, cudaStream_t st) {
+    FaArgs a = {};
+    const bool prefill = c.causal_start >= 0;
+    a.out = (__nv_bfloat16*)c.out; a.q = (const __nv_bfloat16*)c.q; a.k = (const __nv_bfloat16*)c.k; a.v = (const __nv_bfloat16*)c.v;
+    a.n_heads = c.n_heads; a.n_kv = c.n_kv; a.R = c.n_heads / c.n_kv;
+    a.dim = c.hd; a.vdim = c.vhd > 0 ? c.vhd : c.hd;
+    a.ldq = c.ldq > 0 ? c.ldq : c.n_heads * a.dim; a.ldo = c.ldo > 0 ? c.ldo : c.n_heads * a.vdim;
+    a.ldk = c.n_kv * a.dim; a.ldv = c.n_kv * a.vdim;
+    a.n_tokens = c.batch; a.start = c.causal_start; a.seq_len = c.seq_len; a.d_pos = c.d_pos;
+    a.scale = c.scale; a.sink = c.sink; a.qt_coef = c.qt_coef; a.qt_every = c.qt_every;
+    a.row_blocks = (a.R + 15) / 16;
+    if (prefill ? a.n_tokens <= 0 : (!a.d_pos && a.seq_len <= 0)) return set_error(JB_ERR_ARG, "bf16 attention: no tokens or keys");
+    if (!prefill) {
+        a.n_splits = c.n_splits > 0 ? c.n_splits : a.d_pos ? 1 : attn_bf16_splits(a.seq_len, a.n_heads, a.n_kv);
+        if (a.n_splits > 1) {
+            if (a.n_kv * a.row_blocks > ATTN_TICKET_WORDS) return set_error(JB_ERR_LIMIT, "bf16 attention: %d blocks of heads", a.n_kv * a.row_blocks);
+            cudaStreamCaptureStatus cs = cudaStreamCaptureStatusNone;
+            if (cudaStreamIsCapturing(st, &cs) != cudaSuccess) cudaGetLastError();
+            a.part = splitk_buffer((size_t)a.n_heads * a.n_splits * (a.vdim + 2), cs == cudaStreamCaptureStatusNone);
+            a.tickets = ctx() ? ctx()->attn_tickets : nullptr;
+            if (!a.part || !a.tickets) return set_error(JB_ERR_NOMEM, "bf16 attention: partials of %d slices", a.n_splits);
+        }
+    }
+    const int big = a.dim > a.vdim ? a.dim : a.vdim;
+    return big <= 64 ? fa_launch<64>(a, prefill, st) : big <= 128 ? fa_launch<128>(a, prefill, st) : fa_launch<256>(a, prefill, st);
+}
+
+}  // namespace jb

@@ -1,5 +1,6 @@
-// attention_general.cuh — the general attention slice: one query head against keys [kv0, kv1) of an FP16 or INT8
-// cache of any head size up to 512, optional sliding window, cache slot stride >= head size.
+// attention_general.cuh — the general attention slice: one query head against keys [kv0, kv1) of an FP16, INT8, BF16 or
+// FP32 cache of any head size up to 512 (values may have their own), optional sliding window, cache slot stride >= head
+// size, optional softmax sink (one more term in the denominator, no key and no value).
 //
 // Same mathematics as the reference's decode / split-K / prefill kernels (src/kernels/attention.cu:244-375, :382-514,
 // :837-941: s_j = scale * q . k_j with k = k8 * ks for INT8, online softmax, o = Σ p_j v_j with v = v8 * vs), arranged
@@ -8,8 +9,9 @@
 // no CTA-wide barrier per tile — and the warps' states are merged once through shared memory at the end.
 // Used by the general kernels of attention.cu and by the allocation-free entry point.
 #pragma once
-#include "common.cuh"
+#include "layernorm.cuh"
 #include <cfloat>
+#include <type_traits>
 
 namespace jb {
 
@@ -17,57 +19,64 @@ constexpr int AG_WARPS = 4;
 constexpr int AG_THREADS = AG_WARPS * 32;
 constexpr int AG_MAXD = 16;                 // dims per lane: head sizes up to 512
 
-struct AgCache { const void* k; const void* v; const float* ks; const float* vs; int n_kv, chd, kv_int8, window; };
+// kv_kind: EK_F16, EK_INT8 (with scales ks / vs), EK_BF16 or EK_F32.  vhd: value head size (slots of the value cache are
+// vhd wide; 0 = the keys' size and slot stride).
+struct AgCache { const void* k; const void* v; const float* ks; const float* vs; int n_kv, chd, kv_kind, window, vhd = 0; };
 
 inline size_t ag_smem_bytes(int hd) { return (size_t)AG_WARPS * (hd + 2) * sizeof(float); }
 
-// Runs on all AG_THREADS threads of the CTA.  On return M and L hold the slice's running maximum and sum (the same
-// on every thread; M = -FLT_MAX for an empty slice) and emit(d, acc_d) has been called once per dimension d with the
-// unnormalised output, each d by exactly one thread.  `sm` = ag_smem_bytes(hd) of shared memory.
-template <class Emit>
-__device__ __forceinline__ void ag_slice(const __half* q, const AgCache& c, int kvh, int hd, int seq, int kv0, int kv1, float scale,
+__device__ __forceinline__ float to_f32(__half v) { return __half2float(v); }
+template <> __device__ __forceinline__ __half from_f32<__half>(float v) { return __float2half_rn(v); }
+// element d of a cache row of type CT (INT8 rows carry a scale)
+template <typename CT> __device__ __forceinline__ float ag_elem(const char* row, int d, float) { return to_f32(reinterpret_cast<const CT*>(row)[d]); }
+template <> __device__ __forceinline__ float ag_elem<int8_t>(const char* row, int d, float sc) { return (float)reinterpret_cast<const int8_t*>(row)[d] * sc; }
+// Factor on the scores of the query at position p: 1 + coef * ln(floor((p + 1) / every) + 1); every <= 0: none.
+__device__ __forceinline__ float q_temp_factor(int p, float coef, double every) {
+    return every > 0.0 ? 1.0f + coef * logf((float)(floor((double)(p + 1) / every) + 1.0)) : 1.0f;
+}
+// Weight of the accumulated outputs when the softmax has running maximum M, running sum L and an optional sink logit.
+__device__ __forceinline__ float sink_norm(float M, float L, const float* sink) {
+    if (!sink) return L > 0.f ? 1.0f / L : 0.f;
+    if (!(L > 0.f)) return 0.f;
+    const float top = fmaxf(M, *sink), e = expf(M - top);
+    return e / (L * e + expf(*sink - top));
+}
+
+template <typename CT, typename QT, class Emit>
+__device__ __forceinline__ void ag_slice_typed(const QT* q, const AgCache& c, int kvh, int hd, int seq, int kv0, int kv1, float scale,
                                          float* sm, float& M, float& L, Emit emit) {
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const size_t row = (size_t)c.n_kv * c.chd, off = (size_t)kvh * c.chd;
+    const int vhd = c.vhd > 0 ? c.vhd : hd, vslot = c.vhd > 0 ? c.vhd : c.chd;
+    constexpr size_t es = sizeof(CT);
+    const bool scaled = es == 1;
+    const size_t krow = (size_t)c.n_kv * c.chd * es, koff = (size_t)kvh * c.chd * es, vrow = (size_t)c.n_kv * vslot * es, voff = (size_t)kvh * vslot * es;
     float qr[AG_MAXD], acc[AG_MAXD];
     #pragma unroll
-    for (int i = 0; i < AG_MAXD; ++i) { const int d = lane + 32 * i; qr[i] = d < hd ? __half2float(q[d]) : 0.f; acc[i] = 0.f; }
+    for (int i = 0; i < AG_MAXD; ++i) { const int d = lane + 32 * i; qr[i] = d < hd ? to_f32(q[d]) : 0.f; acc[i] = 0.f; }
     float m = -FLT_MAX, l = 0.f;
     const int first = c.window > 0 ? max(kv0, seq - c.window) : kv0;      // keys before the window contribute nothing
     for (int p = first + warp; p < kv1; p += AG_WARPS) {
         float kd[AG_MAXD], dot = 0.f;
-        if (c.kv_int8) {
-            const int8_t* kr = reinterpret_cast<const int8_t*>(c.k) + (size_t)p * row + off;
-            const float sc = c.ks ? c.ks[(size_t)p * c.n_kv + kvh] : 1.0f;
-            #pragma unroll
-            for (int i = 0; i < AG_MAXD; ++i) { const int d = lane + 32 * i; kd[i] = d < hd ? (float)kr[d] * sc : 0.f; }
-        } else {
-            const __half* kr = reinterpret_cast<const __half*>(c.k) + (size_t)p * row + off;
-            #pragma unroll
-            for (int i = 0; i < AG_MAXD; ++i) { const int d = lane + 32 * i; kd[i] = d < hd ? __half2float(kr[d]) : 0.f; }
-        }
+        const char* kr = reinterpret_cast<const char*>(c.k) + (size_t)p * krow + koff;
+        const float ksc = scaled && c.ks ? c.ks[(size_t)p * c.n_kv + kvh] : 1.0f;
+        #pragma unroll
+        for (int i = 0; i < AG_MAXD; ++i) { const int d = lane + 32 * i; kd[i] = d < hd ? ag_elem<CT>(kr, d, ksc) : 0.f; }
         #pragma unroll
         for (int i = 0; i < AG_MAXD; ++i) dot += qr[i] * kd[i];
         const float s = warp_sum(dot) * scale;
         const float m_new = fmaxf(m, s), corr = expf(m - m_new), pw = expf(s - m_new);
         m = m_new;
         l = l * corr + pw;
-        if (c.kv_int8) {
-            const int8_t* vr = reinterpret_cast<const int8_t*>(c.v) + (size_t)p * row + off;
-            const float sc = c.vs ? c.vs[(size_t)p * c.n_kv + kvh] : 1.0f;
-            #pragma unroll
-            for (int i = 0; i < AG_MAXD; ++i) { const int d = lane + 32 * i; if (d < hd) acc[i] = acc[i] * corr + pw * ((float)vr[d] * sc); }
-        } else {
-            const __half* vr = reinterpret_cast<const __half*>(c.v) + (size_t)p * row + off;
-            #pragma unroll
-            for (int i = 0; i < AG_MAXD; ++i) { const int d = lane + 32 * i; if (d < hd) acc[i] = acc[i] * corr + pw * __half2float(vr[d]); }
-        }
+        const char* vr = reinterpret_cast<const char*>(c.v) + (size_t)p * vrow + voff;
+        const float vsc = scaled && c.vs ? c.vs[(size_t)p * c.n_kv + kvh] : 1.0f;
+        #pragma unroll
+        for (int i = 0; i < AG_MAXD; ++i) { const int d = lane + 32 * i; if (d < vhd) acc[i] = acc[i] * corr + pw * ag_elem<CT>(vr, d, vsc); }
     }
     // merge the warps' states
-    float* sm_m = sm; float* sm_l = sm + AG_WARPS; float* sm_o = sm + 2 * AG_WARPS;     // [warp][hd]
+    float* sm_m = sm; float* sm_l = sm + AG_WARPS; float* sm_o = sm + 2 * AG_WARPS;     // [warp][vhd]
     if (lane == 0) { sm_m[warp] = m; sm_l[warp] = l; }
     #pragma unroll
-    for (int i = 0; i < AG_MAXD; ++i) { const int d = lane + 32 * i; if (d < hd) sm_o[warp * hd + d] = acc[i]; }
+    for (int i = 0; i < AG_MAXD; ++i) { const int d = lane + 32 * i; if (d < vhd) sm_o[warp * vhd + d] = acc[i]; }
     __syncthreads();
     M = -FLT_MAX;
     #pragma unroll
@@ -76,25 +85,39 @@ __device__ __forceinline__ void ag_slice(const __half* q, const AgCache& c, int 
     L = 0.f;
     #pragma unroll
     for (int w = 0; w < AG_WARPS; ++w) { e[w] = sm_l[w] > 0.f ? expf(sm_m[w] - M) : 0.f; L += sm_l[w] * e[w]; }
-    for (int d = tid; d < hd; d += AG_THREADS) {
+    for (int d = tid; d < vhd; d += AG_THREADS) {
         float o = 0.f;
         #pragma unroll
-        for (int w = 0; w < AG_WARPS; ++w) o += sm_o[w * hd + d] * e[w];
+        for (int w = 0; w < AG_WARPS; ++w) o += sm_o[w * vhd + d] * e[w];
         emit(d, o);
     }
 }
 
-// out = Σ_s acc_s e^{m_s-M} / Σ_s l_s e^{m_s-M} over the partial records (m, l, acc[hd]) of one head (reference :944-969)
-__device__ __forceinline__ void ag_merge_slices(__half* out, const float* pb, int hd, int n_splits) {
+// Runs on all AG_THREADS threads of the CTA.  On return M and L hold the slice's running maximum and sum (the same
+// on every thread; M = -FLT_MAX for an empty slice) and emit(d, acc_d) has been called once per dimension d with the
+// unnormalised output, each d by exactly one thread.  `sm` = ag_smem_bytes(hd) of shared memory.
+template <typename QT, class Emit>
+__device__ __forceinline__ void ag_slice(const QT* q, const AgCache& c, int kvh, int hd, int seq, int kv0, int kv1, float scale,
+                                         float* sm, float& M, float& L, Emit emit) {
+    // fp16 queries go with an FP16 or INT8 cache, BF16 and FP32 queries with a cache of their own type
+    if constexpr (sizeof(QT) == 2 && !std::is_same<QT, __nv_bfloat16>::value) {
+        if (c.kv_kind == EK_INT8) { ag_slice_typed<int8_t>(q, c, kvh, hd, seq, kv0, kv1, scale, sm, M, L, emit); return; }
+    }
+    ag_slice_typed<QT>(q, c, kvh, hd, seq, kv0, kv1, scale, sm, M, L, emit);
+}
+
+// out = Σ_s acc_s e^{m_s-M} / (Σ_s l_s e^{m_s-M} [+ e^{sink-M}]) over the partial records (m, l, acc[hd]) of one head (reference :944-969)
+template <typename OT>
+__device__ __forceinline__ void ag_merge_slices(OT* out, const float* pb, int hd, int n_splits, const float* sink = nullptr) {
     float M = -FLT_MAX;
     for (int s = 0; s < n_splits; ++s) M = fmaxf(M, pb[(size_t)s * (hd + 2)]);
     float L = 0.f;
     for (int s = 0; s < n_splits; ++s) L += pb[(size_t)s * (hd + 2) + 1] * expf(pb[(size_t)s * (hd + 2)] - M);
-    const float inv = L > 0.f ? 1.0f / L : 0.f;
+    const float inv = sink_norm(M, L, sink);
     for (int d = threadIdx.x; d < hd; d += blockDim.x) {
         float acc = 0.f;
         for (int s = 0; s < n_splits; ++s) acc += pb[(size_t)s * (hd + 2) + 2 + d] * expf(pb[(size_t)s * (hd + 2)] - M);
-        out[d] = __float2half_rn(acc * inv);
+        out[d] = from_f32<OT>(acc * inv);
     }
 }
 

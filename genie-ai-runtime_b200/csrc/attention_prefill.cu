@@ -323,7 +323,7 @@ int launch_attention_prefill_fast(const AttnCall& c, cudaStream_t st) {
     alignas(64) CUtensorMap kmap, vmap;
     if (!attn_tma_encode(&kmap, c.k, rows, c.n_kv) || !attn_tma_encode(&vmap, c.v, rows, c.n_kv))
         return set_error(JB_ERR_CUDA, "prefill attention: tensor map for the KV cache refused");
-    ApArgs a = { c.out, c.q, c.ks, c.vs, c.n_heads, c.n_kv, N, c.causal_start, c.scale, cx->d_status };
+    ApArgs a = { (__half*)c.out, (const __half*)c.q, c.ks, c.vs, c.n_heads, c.n_kv, N, c.causal_start, c.scale, cx->d_status };
     const int G = c.n_heads / c.n_kv;
     auto kern = G == 4 ? attn_prefill_kernel<4> : (G == 2 ? attn_prefill_kernel<2> : attn_prefill_kernel<1>);
     const int gi = G == 4 ? 2 : (G == 2 ? 1 : 0);

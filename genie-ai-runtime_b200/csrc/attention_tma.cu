@@ -459,7 +459,7 @@ int launch_attention_tma(const AttnCall& c, cudaStream_t st) {
     int n_splits = c.n_splits > 0 ? c.n_splits : am_splits(rows > 0 ? rows : 1, c.n_kv, batch, cx->sm_count);
     if (n_splits > 64) n_splits = 64;                       // the merge holds one slice per thread of the last CTA
     AmArgs a = {};
-    a.out = c.out; a.q = c.q; a.ks = c.ks; a.vs = c.vs;
+    a.out = (__half*)c.out; a.q = (const __half*)c.q; a.ks = c.ks; a.vs = c.vs;
     a.ragged = c.tma_maps ? 1 : 0; a.ks_list = c.ks_list; a.vs_list = c.vs_list; a.seq_lens = c.seq_lens;
     a.n_heads = c.n_heads; a.n_kv = c.n_kv; a.seq_len = c.seq_len; a.d_pos = c.d_pos; a.scale = c.scale; a.status = cx->d_status;
     static const bool nocompute = getenv("JLLM_B200_ATTN_NOCOMPUTE") != nullptr;

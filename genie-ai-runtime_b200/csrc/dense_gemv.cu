@@ -1,0 +1,203 @@
+// dense_gemv.cu — one token against dense weights: the decode products of layer-list models, HBM-bound.
+//
+// Two CTAs of eight warps per SM; the output rows (or gate / up row pairs) are dealt to the warps in contiguous runs, a
+// warp walks R rows at a time and keeps eight 16-byte weight loads per lane in flight, one batch ahead of the arithmetic.
+// Where the rows do not depend on the previous kernel (all modes but the expert ones) the first batch is requested before
+// griddepcontrol.wait, so the weights stream in while the input vector is still being produced and normed.  The input
+// vector is held in shared memory in the activation type (what the prompt path multiplies), sums are fp32.
+#include "dense.cuh"
+
+namespace jb {
+
+constexpr int DG_THREADS = 256, DG_WARPS = DG_THREADS / 32, DG_LOADS = 8;
+
+__device__ __forceinline__ float dot16(uint4 w, uint4 h, float acc, float) {
+    acc = fmaf(__uint_as_float(w.x), __uint_as_float(h.x), acc); acc = fmaf(__uint_as_float(w.y), __uint_as_float(h.y), acc);
+    acc = fmaf(__uint_as_float(w.z), __uint_as_float(h.z), acc); return fmaf(__uint_as_float(w.w), __uint_as_float(h.w), acc);
+}
+__device__ __forceinline__ float dot16(uint4 w, uint4 h, float acc, __nv_bfloat16) {
+    const uint32_t ww[4] = {w.x, w.y, w.z, w.w}, hh[4] = {h.x, h.y, h.z, h.w};
+    #pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        acc = fmaf(__uint_as_float(ww[i] << 16), __uint_as_float(hh[i] << 16), acc);
+        acc = fmaf(__uint_as_float(ww[i] & 0xFFFF0000u), __uint_as_float(hh[i] & 0xFFFF0000u), acc);
+    }
+    return acc;
+}
+
+struct DgArgs {
+    DenseGemv g;
+    int nchunk;          // 16-byte chunks of the input vector (of one expert's input for GEMV_MOE_DOWN)
+    uint32_t magic;      // ceil(2^32 / nchunk): chunk / nchunk by one multiply
+};
+
+template <typename T, int MODE, int R>
+__global__ void __launch_bounds__(DG_THREADS, 2) dense_gemv_kernel(const DgArgs p) {
+    constexpr int U = DG_LOADS / R;              // chunks per row in a batch
+    extern __shared__ __align__(16) unsigned char dg_sm[];
+    __shared__ float red[DG_WARPS];
+    __shared__ int s_ids[MOE_MAX_TOP];
+    __shared__ float s_wts[MOE_MAX_TOP];
+    const DenseGemv& g = p.g;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int total_warps = gridDim.x * DG_WARPS, wid = blockIdx.x * DG_WARPS + warp;
+    const int items = MODE == GEMV_MOE_UP ? g.route.top * g.M : g.M;
+    const int r0 = (int)((long long)items * wid / total_warps), r1 = (int)((long long)items * (wid + 1) / total_warps);
+    constexpr int STEP = MODE == GEMV_MOE_UP ? 1 : R;                 // items per group (an up item is two rows)
+    const int nchunk = MODE == GEMV_MOE_DOWN ? p.nchunk * g.route.top : p.nchunk;
+    const int nb = (nchunk + 32 * U - 1) / (32 * U);
+    const int n_batches = r1 > r0 ? ((r1 - r0 + STEP - 1) / STEP) * nb : 0;
+    uint4* hs = reinterpret_cast<uint4*>(dg_sm);
+
+    auto load = [&](int item, int b, uint4 (&w)[DG_LOADS]) {
+        #pragma unroll
+        for (int r = 0; r < R; ++r) {
+            const uint4* row = nullptr;
+            if (MODE == GEMV_MOE_UP) {
+                const int k = item / g.M, f = item - k * g.M;
+                row = reinterpret_cast<const uint4*>(r == 0 ? g.W : g.W_up) + ((size_t)s_ids[k] * g.M + f) * p.nchunk;
+            } else if (MODE != GEMV_MOE_DOWN) {
+                row = reinterpret_cast<const uint4*>(g.W) + (size_t)min(item + r, r1 - 1) * p.nchunk;
+            }
+            #pragma unroll
+            for (int u = 0; u < U; ++u) {
+                const int c = (b * U + u) * 32 + lane;
+                w[r * U + u] = make_uint4(0, 0, 0, 0);
+                if (c < nchunk) {
+                    if (MODE == GEMV_MOE_DOWN) {
+                        const int k = p.nchunk == 1 ? c : (int)__umulhi((uint32_t)c, p.magic), cc = c - k * p.nchunk;
+                        w[r * U + u] = __ldg(reinterpret_cast<const uint4*>(g.W) + ((size_t)s_ids[k] * g.M + min(item + r, r1 - 1)) * p.nchunk + cc);
+                    } else {
+                        w[r * U + u] = __ldg(row + c);
+                    }
+                }
+            }
+        }
+    };
+
+    uint4 cur[DG_LOADS], nxt[DG_LOADS];
+    if (MODE == GEMV_NORM || MODE == GEMV_PLAIN) { if (n_batches > 0) load(r0, 0, cur); }
+    pdl_wait();
+    pdl_launch();
+    // ── the input vector ──
+    if (MODE == GEMV_NORM) {
+        float* buf = reinterpret_cast<float*>(dg_sm + (size_t)p.nchunk * 16);
+        T* h = reinterpret_cast<T*>(hs);
+        norm_step_row<T, DG_THREADS>(g.norm, 0, buf, red, blockIdx.x == 0 && g.norm.x_out, h);
+        __syncthreads();
+        if (blockIdx.x == 0 && g.norm.h)
+            for (int i = threadIdx.x; i < p.nchunk; i += DG_THREADS) reinterpret_cast<uint4*>(g.norm.h)[i] = hs[i];
+    } else {
+        for (int i = threadIdx.x; i < nchunk; i += DG_THREADS) hs[i] = reinterpret_cast<const uint4*>(g.x)[i];
+        if (MODE == GEMV_MOE_UP) {
+            if (warp == 0) {
+                float* c = reinterpret_cast<float*>(dg_sm + (size_t)nchunk * 16);
+                moe_route_warp(g.z, g.route, c, c + g.route.n_experts, c + 2 * g.route.n_experts, [&](int k, int id, float w) {
+                    s_ids[k] = id; s_wts[k] = w;
+                    if (blockIdx.x == 0) { g.ids[k] = id; g.wts[k] = w; }
+                });
+            }
+        } else if (MODE == GEMV_MOE_DOWN) {
+            for (int k = threadIdx.x; k < g.route.top; k += DG_THREADS) { s_ids[k] = g.ids[k]; s_wts[k] = g.wts[k]; }
+        }
+        __syncthreads();
+        if (MODE != GEMV_PLAIN && n_batches > 0) load(r0, 0, cur);
+    }
+    // ── the products ──
+    float acc[R];
+    #pragma unroll
+    for (int r = 0; r < R; ++r) acc[r] = 0.f;
+    int item = r0, b = 0;
+    for (int it = 0; it < n_batches; ++it) {
+        int item_n = item, b_n = b + 1;
+        if (b_n == nb) { b_n = 0; item_n += STEP; }
+        if (it + 1 < n_batches) load(item_n, b_n, nxt);
+        #pragma unroll
+        for (int u = 0; u < U; ++u) {
+            const int c = (b * U + u) * 32 + lane;
+            if (c < nchunk) {
+                const uint4 h = hs[c];
+                if (MODE == GEMV_MOE_DOWN) {
+                    const float w = s_wts[p.nchunk == 1 ? c : (int)__umulhi((uint32_t)c, p.magic)];
+                    #pragma unroll
+                    for (int r = 0; r < R; ++r) acc[r] = fmaf(w, dot16(cur[r * U + u], h, 0.f, T()), acc[r]);
+                } else {
+                    #pragma unroll
+                    for (int r = 0; r < R; ++r) acc[r] = dot16(cur[r * U + u], h, acc[r], T());
+                }
+            }
+        }
+        if (b_n == 0) {
+            #pragma unroll
+            for (int r = 0; r < R; ++r) acc[r] = warp_sum(acc[r]);
+            if (MODE == GEMV_MOE_UP) {
+                if (lane == 0) {
+                    const int k = item / g.M, f = item - k * g.M;
+                    reinterpret_cast<T*>(g.seg[0].y)[(long long)k * g.seg[0].ld + f] = from_f32<T>(silu_f(acc[0]) * acc[R > 1 ? 1 : 0]);
+                }
+            } else {
+                #pragma unroll
+                for (int r = 0; r < R; ++r)
+                    if (lane == r && item + r < r1) store_seg<T>(g.seg, g.nseg, g.softcap, g.d_pos, 0, item + r, acc[r]);
+            }
+            #pragma unroll
+            for (int r = 0; r < R; ++r) acc[r] = 0.f;
+        }
+        #pragma unroll
+        for (int i = 0; i < DG_LOADS; ++i) cur[i] = nxt[i];
+        item = item_n; b = b_n;
+    }
+}
+
+template <typename T, int MODE, int R>
+static int dg_go(const DgArgs& p, int grid, size_t smem, cudaStream_t st) {
+    static size_t set = 48 * 1024;
+    if (smem > set) {
+        JB_CUDA(cudaFuncSetAttribute(dense_gemv_kernel<T, MODE, R>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        set = smem;
+    }
+    JB_CUDA(launch_k(dense_gemv_kernel<T, MODE, R>, dim3(grid), dim3(DG_THREADS), smem, st, pdl_enabled(), p));
+    count_launch();
+    return JB_OK;
+}
+template <typename T, int MODE>
+static int dg_rows(const DgArgs& p, int R, int grid, size_t smem, cudaStream_t st) {
+    if constexpr (MODE == GEMV_MOE_UP) return dg_go<T, MODE, 2>(p, grid, smem, st);
+    else return R == 4 ? dg_go<T, MODE, 4>(p, grid, smem, st) : R == 2 ? dg_go<T, MODE, 2>(p, grid, smem, st) : dg_go<T, MODE, 1>(p, grid, smem, st);
+}
+template <typename T>
+static int dg_mode(const DgArgs& p, int R, int grid, size_t smem, cudaStream_t st) {
+    switch (p.g.mode) {
+        case GEMV_NORM:   return dg_rows<T, GEMV_NORM>(p, R, grid, smem, st);
+        case GEMV_PLAIN:  return dg_rows<T, GEMV_PLAIN>(p, R, grid, smem, st);
+        case GEMV_MOE_UP: return dg_rows<T, GEMV_MOE_UP>(p, R, grid, smem, st);
+        default:          return dg_rows<T, GEMV_MOE_DOWN>(p, R, grid, smem, st);
+    }
+}
+
+int launch_dense_gemv(const DenseGemv& a, cudaStream_t st) {
+    DeviceCtx* c = ctx();
+    if (!c) return set_error(JB_ERR_STATE, "dense gemv: library not initialised");
+    if (a.M <= 0 || a.K <= 0) return set_error(JB_ERR_ARG, "dense gemv: M=%d K=%d", a.M, a.K);
+    if (!a.W || (a.mode != GEMV_NORM && !a.x) || (a.mode == GEMV_MOE_UP && (!a.W_up || !a.z)) || (a.mode >= GEMV_MOE_UP && (!a.ids || !a.wts)))
+        return set_error(JB_ERR_PTR, "dense gemv: null pointer");
+    if (a.mode >= GEMV_MOE_UP && (a.route.top <= 0 || a.route.top > MOE_MAX_TOP || a.route.n_experts > MOE_MAX_EXPERTS)) return set_error(JB_ERR_LIMIT, "dense gemv: top %d of %d experts", a.route.top, a.route.n_experts);
+    DgArgs p;
+    p.g = a;
+    const int es = a.kind == EK_F32 ? 4 : 2;
+    p.nchunk = pad8(a.K) * es / 16;
+    p.magic = p.nchunk > 1 ? (uint32_t)((0x100000000ull + p.nchunk - 1) / p.nchunk) : 0;
+    const int chunks = a.mode == GEMV_MOE_DOWN ? p.nchunk * a.route.top : p.nchunk;
+    size_t smem = (size_t)chunks * 16;
+    if (a.mode == GEMV_NORM) smem += (size_t)pad8(a.K) * 4;
+    if (a.mode == GEMV_MOE_UP) smem += (size_t)(2 * a.route.n_experts + a.route.n_groups) * 4;
+    if (smem > (size_t)c->max_smem_optin - 2048) return set_error(JB_ERR_LIMIT, "dense gemv: input of %d elements", a.K);
+    const int items = a.mode == GEMV_MOE_UP ? a.route.top * a.M : a.M;
+    const int full = 2 * c->sm_count, per_warp = items / (full * DG_WARPS);
+    const int R = per_warp >= 4 ? 4 : per_warp >= 2 ? 2 : 1;
+    const int want = (items + DG_WARPS - 1) / DG_WARPS;
+    const int grid = want < full ? want : full;
+    return a.kind == EK_F32 ? dg_mode<float>(p, R, grid, smem, st) : dg_mode<__nv_bfloat16>(p, R, grid, smem, st);
+}
+
+}  // namespace jb

@@ -1,0 +1,64 @@
+// dense_simt.cu — dense products over many tokens on the CUDA cores, in true fp32 (FFMA, no reduced-precision matrix mode):
+// the 32-bit path of layer-list models.  64 x 64 output tiles, 4 x 4 per thread, K tiles of 16; groups (experts) on grid.z.
+#include "dense.cuh"
+
+namespace jb {
+
+constexpr int DS_T = 64, DS_K = 16, DS_THREADS = 256;
+
+template <bool GLU>
+__global__ void __launch_bounds__(DS_THREADS) dense_simt_kernel(const DenseGemm a) {
+    pdl_wait();
+    __shared__ float ws[DS_K][DS_T + 4], us[GLU ? DS_K : 1][DS_T + 4], xs[DS_K][DS_T + 4];
+    const int grp = blockIdx.z, t_lo = a.off ? a.off[grp] : 0, t_hi = a.off ? a.off[grp + 1] : a.N;
+    const int t0 = t_lo + blockIdx.y * DS_T, r0 = blockIdx.x * DS_T, ld = pad8(a.K);
+    if (t0 >= t_hi) return;
+    const float* W = reinterpret_cast<const float*>(a.W) + (size_t)grp * a.M * ld;
+    const float* V = GLU ? reinterpret_cast<const float*>(a.W_up) + (size_t)grp * a.M * ld : nullptr;
+    const float* x = reinterpret_cast<const float*>(a.x);
+    const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;       // thread: rows 4 tx .. , tokens 4 ty ..
+    float acc[4][4] = {}, acu[4][4] = {};
+    for (int k0 = 0; k0 < a.K; k0 += DS_K) {
+        for (int i = threadIdx.x; i < DS_T * DS_K; i += DS_THREADS) {
+            const int k = i % DS_K, j = i / DS_K;
+            const bool kin = k0 + k < a.K;
+            ws[k][j] = kin && r0 + j < a.M ? W[(size_t)(r0 + j) * ld + k0 + k] : 0.f;
+            if (GLU) us[k][j] = kin && r0 + j < a.M ? V[(size_t)(r0 + j) * ld + k0 + k] : 0.f;
+            xs[k][j] = kin && t0 + j < t_hi ? x[(size_t)(t0 + j) * ld + k0 + k] : 0.f;
+        }
+        __syncthreads();
+        #pragma unroll
+        for (int k = 0; k < DS_K; ++k) {
+            float w[4], u[4], v[4];
+            #pragma unroll
+            for (int i = 0; i < 4; ++i) { w[i] = ws[k][4 * tx + i]; u[i] = GLU ? us[k][4 * tx + i] : 0.f; v[i] = xs[k][4 * ty + i]; }
+            #pragma unroll
+            for (int i = 0; i < 4; ++i)
+                #pragma unroll
+                for (int j = 0; j < 4; ++j) { acc[i][j] = fmaf(w[i], v[j], acc[i][j]); if (GLU) acu[i][j] = fmaf(u[i], v[j], acu[i][j]); }
+        }
+        __syncthreads();
+    }
+    #pragma unroll
+    for (int j = 0; j < 4; ++j)
+        #pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int r = r0 + 4 * tx + i, t = t0 + 4 * ty + j;
+            if (r < a.M && t < t_hi) store_seg<float>(a.seg, a.nseg, a.softcap, nullptr, t, r, GLU ? silu_f(acc[i][j]) * acu[i][j] : acc[i][j]);
+        }
+}
+
+int launch_dense_gemm_simt(const DenseGemm& a, cudaStream_t st) {
+    if (a.N <= 0 || a.M <= 0) return JB_OK;
+    if (a.kind != EK_F32) return set_error(JB_ERR_TYPE, "dense fp32 gemm: element kind %d", a.kind);
+    if (!a.W || !a.x || (a.swiglu && !a.W_up) || (a.n_groups > 1 && !a.off)) return set_error(JB_ERR_PTR, "dense fp32 gemm: null pointer");
+    const dim3 grid((a.M + DS_T - 1) / DS_T, (a.N + DS_T - 1) / DS_T, a.n_groups);
+    if (grid.y > 65535) return set_error(JB_ERR_LIMIT, "dense fp32 gemm: %d tokens", a.N);
+    if (a.swiglu) JB_CUDA(launch_k(dense_simt_kernel<true>, grid, dim3(DS_THREADS), 0, st, pdl_enabled(), a));
+    else          JB_CUDA(launch_k(dense_simt_kernel<false>, grid, dim3(DS_THREADS), 0, st, pdl_enabled(), a));
+    count_launch();
+    return JB_OK;
+}
+int launch_dense_gemm(const DenseGemm& a, cudaStream_t st) { return a.kind == EK_F32 ? launch_dense_gemm_simt(a, st) : launch_dense_gemm_tc(a, st); }
+
+}  // namespace jb

@@ -1,0 +1,238 @@
+// dense_tc.cu — dense bf16 products over many tokens on the 5th-generation tensor cores: tcgen05.mma with both operands
+// brought by TMA and the accumulator in tensor memory.  One weight matrix, or one per group (the experts of a mixture over
+// their own token rows), optionally a gate / up pair with SwiGLU on the way out.
+//
+// One persistent CTA per SM walks 128 (weight rows) x n_tile (tokens) output tiles, K tiles of 64, four operand stages of
+// 48 KB (128 x 64 weights + up to 256 x 64 tokens; for a pair two weight tiles + up to 128 tokens), two accumulators in
+// tensor memory so that the drain of one tile overlaps the K loop of the next.  Weight rows are the M side, so a handful
+// of tokens needs only a narrow N.  Warps: 0 TMA producer, 1 MMA issuer, 2-3 idle, 4-7 drain (their index modulo 4 is the
+// tensor-memory lane quarter they may read).  Tiles of a group never mix with another's: the token box of a group's last
+// tile reads on into the next group's rows, and the drain stores only its own.  Every mbarrier wait is bounded.
+#include "dense.cuh"
+#include "tc.cuh"
+
+namespace jb {
+
+constexpr int DT_M = 128, DT_K = 64, DT_STAGES = 4, DT_THREADS = 256;
+constexpr int DT_STAGE_BYTES = 48 * 1024;
+constexpr int DT_SMEM = DT_STAGES * DT_STAGE_BYTES + 1024;
+constexpr int DT_MAX_GROUPS = MOE_MAX_EXPERTS;
+
+struct DtArgs {
+    OutSeg seg[3]; int nseg;
+    int M, N, n_tile, k_tiles, n_groups;
+    float softcap;
+    const int* off;
+    int* status;
+};
+
+// GLU: two weight maps (gate, up), two accumulators side by side per buffer
+template <bool GLU>
+__global__ void __launch_bounds__(DT_THREADS, 1) dense_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_constant__ CUtensorMap umap,
+                                                                 const __grid_constant__ CUtensorMap xmap, const DtArgs a) {
+    extern __shared__ uint8_t dt_smem_raw[];
+    __shared__ uint64_t full[DT_STAGES], empty[DT_STAGES], acc_full[2], acc_empty[2], drain_bar;
+    __shared__ uint32_t tmem_slot;
+    __shared__ volatile int fail;
+    __shared__ int t_first[DT_MAX_GROUPS + 1];       // tiles before each group
+    __shared__ int row_off[DT_MAX_GROUPS + 1];       // first token row of each group
+    uint8_t* smem = dt_smem_raw + ((1024u - (smem_u32(dt_smem_raw) & 1023u)) & 1023u);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    constexpr int A_BYTES = (GLU ? 2 : 1) * DT_M * DT_K * 2;
+    const int tiles_m = (a.M + DT_M - 1) / DT_M;
+
+    if (threadIdx.x == 0) {
+        for (int s = 0; s < DT_STAGES; ++s) { mbar_init(&full[s], 1); mbar_init(&empty[s], 1); }
+        for (int i = 0; i < 2; ++i) { mbar_init(&acc_full[i], 1); mbar_init(&acc_empty[i], 4); }
+        mbar_init(&drain_bar, 1);
+        fence_mbar_init();
+        fail = 0;
+    }
+    if (warp == 1) {
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&tmem_slot)), "r"(512u) : "memory");
+        asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+    }
+    pdl_wait();
+    pdl_launch();
+    if (warp == 2) {                                  // tile counts of the groups, prefix-summed 32 at a time
+        int base = 0;
+        for (int e0 = 0; e0 < a.n_groups; e0 += 32) {
+            const int e = e0 + lane;
+            int lo = 0, hi = 0;
+            if (e < a.n_groups) { lo = a.off ? a.off[e] : 0; hi = a.off ? a.off[e + 1] : a.N; }
+            const int v = ((hi - lo + a.n_tile - 1) / a.n_tile) * tiles_m;
+            int s = v;
+            #pragma unroll
+            for (int o = 1; o < 32; o <<= 1) { const int u = __shfl_up_sync(0xFFFFFFFFu, s, o); if (lane >= o) s += u; }
+            if (e < a.n_groups) { t_first[e] = base + s - v; row_off[e] = lo; if (e + 1 == a.n_groups) row_off[e + 1] = hi; }
+            base += __shfl_sync(0xFFFFFFFFu, s, 31);
+        }
+        if (lane == 0) t_first[a.n_groups] = base;
+    }
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    const uint32_t tmem = tmem_slot;
+    const int n_work = t_first[a.n_groups];
+    int grp = 0;
+    // work item w -> group, weight row tile, first token row (the groups are walked in order; within one, token tiles fastest)
+    auto locate = [&](int w, int& mt, int& n0, int& n_end) {
+        while (w >= t_first[grp + 1]) ++grp;
+        n_end = row_off[grp + 1];
+        const int tn = (n_end - row_off[grp] + a.n_tile - 1) / a.n_tile, i = w - t_first[grp];
+        mt = i / tn;
+        n0 = row_off[grp] + (i - mt * tn) * a.n_tile;
+    };
+
+    if (warp == 0) {
+        if (lane == 0) {
+            uint32_t it = 0;
+            const uint32_t bytes = A_BYTES + (uint32_t)a.n_tile * DT_K * 2;
+            for (int w = blockIdx.x; w < n_work && !fail; w += gridDim.x) {
+                int mt, n0, n_end;
+                locate(w, mt, n0, n_end);
+                const int wrow = grp * a.M + mt * DT_M;
+                for (int t = 0; t < a.k_tiles; ++t, ++it) {
+                    const int s = it % DT_STAGES;
+                    if (!tc_wait(&empty[s], ((it / DT_STAGES) & 1) ^ 1) || fail) { tc_fail(&fail, a.status); break; }
+                    uint8_t* st = smem + s * DT_STAGE_BYTES;
+                    mbar_expect_tx(&full[s], bytes);
+                    tma_load_2d(st, &wmap, t * DT_K, wrow, &full[s]);
+                    if (GLU) tma_load_2d(st + DT_M * DT_K * 2, &umap, t * DT_K, wrow, &full[s]);
+                    tma_load_2d(st + A_BYTES, &xmap, t * DT_K, n0, &full[s]);
+                }
+            }
+        }
+    } else if (warp == 1) {
+        if (lane == 0) {
+            // bf16 x bf16 -> fp32, both operands K-major, M = 128, N = n_tile
+            const uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(a.n_tile >> 3) << 17) | ((uint32_t)(DT_M >> 4) << 24);
+            const uint64_t ad0 = tc_smem_desc(smem_u32(smem)), bd0 = tc_smem_desc(smem_u32(smem + A_BYTES));
+            uint32_t it = 0, j = 0;
+            bool ok = true;
+            for (int w = blockIdx.x; w < n_work && ok; w += gridDim.x, ++j) {
+                const uint32_t d = tmem + (j & 1) * 256u;
+                if (!tc_wait(&acc_empty[j & 1], ((j >> 1) & 1) ^ 1)) { ok = false; break; }
+                tc_fence_after();
+                for (int t = 0; t < a.k_tiles; ++t, ++it) {
+                    const uint32_t s = it % DT_STAGES;
+                    if (!tc_wait(&full[s], (it / DT_STAGES) & 1)) { ok = false; break; }
+                    tc_fence_after();
+                    const uint64_t ad = ad0 + (uint64_t)(s * (DT_STAGE_BYTES >> 4)), bd = bd0 + (uint64_t)(s * (DT_STAGE_BYTES >> 4));
+                    #pragma unroll
+                    for (int k = 0; k < 4; ++k) {
+                        tc_mma_f16(d, ad + 2 * k, bd + 2 * k, idesc, (uint32_t)(t != 0 || k != 0));
+                        if (GLU) tc_mma_f16(d + 128u, ad + ((DT_M * DT_K * 2) >> 4) + 2 * k, bd + 2 * k, idesc, (uint32_t)(t != 0 || k != 0));
+                    }
+                    tc_commit(&empty[s]);
+                }
+                tc_commit(&acc_full[j & 1]);
+            }
+            if (!ok) tc_fail(&fail, a.status);
+            // nothing of this CTA may still be running on the tensor pipe when the columns are freed
+            tc_commit(&drain_bar);
+            tc_wait(&drain_bar, 0);
+        }
+    } else if (warp >= 4) {
+        const int q = warp & 3, rl = q * 32 + lane;
+        uint32_t j = 0;
+        for (int w = blockIdx.x; w < n_work; w += gridDim.x, ++j) {
+            const uint32_t acc = j & 1;
+            int mt, n0, n_end;
+            locate(w, mt, n0, n_end);
+            bool good = true;
+            if (lane == 0) good = tc_wait(&acc_full[acc], (j >> 1) & 1) && !fail;
+            good = __shfl_sync(0xFFFFFFFFu, (int)good, 0) != 0;
+            if (!good) { if (lane == 0) tc_fail(&fail, a.status); break; }
+            tc_fence_after();
+            int row = mt * DT_M + rl, s = 0;
+            const bool in = row < a.M;
+            while (s + 1 < a.nseg && row >= a.seg[s].rows) { row -= a.seg[s].rows; ++s; }
+            const long long ld = a.seg[s].ld;
+            const bool f32 = a.seg[s].f32 != 0;
+            float* yf = reinterpret_cast<float*>(a.seg[s].y) + row;
+            __nv_bfloat16* yb = reinterpret_cast<__nv_bfloat16*>(a.seg[s].y) + row;
+            const int cols = min(a.n_tile, n_end - n0);
+            const uint32_t t_acc = tmem + ((uint32_t)(q * 32) << 16) + acc * 256u;
+            for (int cb = 0; cb < cols; cb += 32) {
+                uint32_t r[32];
+                tc_ld32(t_acc + (uint32_t)cb, r);
+                if (GLU) {
+                    uint32_t u[32];
+                    tc_ld32(t_acc + 128u + (uint32_t)cb, u);
+                    #pragma unroll
+                    for (int c = 0; c < 32; ++c) r[c] = __float_as_uint(silu_f(__uint_as_float(r[c])) * __uint_as_float(u[c]));
+                }
+                if (in) {
+                    #pragma unroll
+                    for (int c = 0; c < 32; ++c) {
+                        if (cb + c < cols) {
+                            float v = __uint_as_float(r[c]);
+                            if (a.softcap > 0.f) v = a.softcap * tanhf(v / a.softcap);
+                            if (f32) yf[(n0 + cb + c) * ld] = v;
+                            else     yb[(n0 + cb + c) * ld] = __float2bfloat16_rn(v);
+                        }
+                    }
+                }
+            }
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) mbar_arrive(&acc_empty[acc]);
+        }
+    }
+    __syncwarp();
+    tc_fence_before();
+    __syncthreads();
+    if (warp == 1) {
+        tc_fence_after();
+        asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(512u) : "memory");
+    }
+}
+
+// Token-tile width: wide tiles use the tensor pipe best, but too few of them leave SMs idle for the last round.
+static int dt_pick(int tiles_m, int tokens_per_group, int groups, int max_tile, int sm) {
+    int best = 32;
+    double cost = 1e30;
+    for (int c = 32; c <= max_tile; c <<= 1) {
+        if (c > 32 && c / 2 >= tokens_per_group) break;
+        const long long tiles = (long long)groups * tiles_m * ((tokens_per_group + c - 1) / c);
+        const double t = (double)((tiles + sm - 1) / sm) * ((c < 128 ? 128 : c) / 256.0 + 0.02);
+        if (t <= cost) { cost = t; best = c; }
+    }
+    return best;
+}
+
+int launch_dense_gemm_tc(const DenseGemm& a, cudaStream_t st) {
+    if (a.N <= 0 || a.M <= 0) return JB_OK;
+    DeviceCtx* c = ctx();
+    if (!c) return set_error(JB_ERR_STATE, "dense gemm: library not initialised");
+    if (a.kind != EK_BF16) return set_error(JB_ERR_TYPE, "dense gemm: element kind %d", a.kind);
+    if (!a.W || !a.x || (a.swiglu && !a.W_up) || (a.n_groups > 1 && !a.off)) return set_error(JB_ERR_PTR, "dense gemm: null pointer");
+    if (a.n_groups < 1 || a.n_groups > DT_MAX_GROUPS || a.K <= 0) return set_error(JB_ERR_LIMIT, "dense gemm: %d groups, K=%d", a.n_groups, a.K);
+    DtArgs p;
+    for (int i = 0; i < 3; ++i) p.seg[i] = a.seg[i];
+    p.nseg = a.nseg; p.M = a.M; p.N = a.N; p.n_groups = a.n_groups; p.softcap = a.softcap; p.off = a.off; p.status = c->d_status;
+    p.k_tiles = (a.K + DT_K - 1) / DT_K;
+    const int tiles_m = (a.M + DT_M - 1) / DT_M, per = (a.N + a.n_groups - 1) / a.n_groups;
+    p.n_tile = dt_pick(tiles_m, per, a.n_groups, a.swiglu ? 128 : 256, c->sm_count);
+    CUtensorMap wm, um, xm;
+    const long long ld = pad8(a.K);
+    if (!encode_tile_map(&wm, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, a.W, (long long)a.n_groups * a.M, a.K, ld, DT_M) ||
+        !encode_tile_map(&um, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, a.swiglu ? a.W_up : a.W, (long long)a.n_groups * a.M, a.K, ld, DT_M) ||
+        !encode_tile_map(&xm, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, a.x, a.N, a.K, ld, p.n_tile))
+        return set_error(JB_ERR_CUDA, "dense gemm: tensor map refused (M=%d N=%d K=%d)", a.M, a.N, a.K);
+    static bool attr = false;
+    if (!attr) {
+        JB_CUDA(cudaFuncSetAttribute(dense_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, DT_SMEM));
+        JB_CUDA(cudaFuncSetAttribute(dense_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, DT_SMEM));
+        attr = true;
+    }
+    const long long bound = (long long)tiles_m * ((a.N + p.n_tile - 1) / p.n_tile + (a.n_groups - 1));
+    const dim3 grid((unsigned)(bound < c->sm_count ? bound : c->sm_count));
+    if (a.swiglu) JB_CUDA(launch_k(dense_tc_kernel<true>, grid, dim3(DT_THREADS), DT_SMEM, st, pdl_enabled(), wm, um, xm, p));
+    else          JB_CUDA(launch_k(dense_tc_kernel<false>, grid, dim3(DT_THREADS), DT_SMEM, st, pdl_enabled(), wm, um, xm, p));
+    count_launch();
+    return JB_OK;
+}
+
+}  // namespace jb

@@ -1,0 +1,32 @@
+// layernorm.cu — the residual step over many rows (prompt path of layer-list models): one CTA per row.
+#include "layernorm.cuh"
+
+namespace jb {
+
+constexpr int NR_THREADS = 256;
+
+template <typename T>
+__global__ void __launch_bounds__(NR_THREADS) norm_rows_kernel(const NormStep a) {
+    pdl_wait();
+    extern __shared__ __align__(16) float nr_buf[];
+    __shared__ float red[NR_THREADS / 32];
+    const int row = blockIdx.x;
+    norm_step_row<T, NR_THREADS>(a, row, nr_buf, red, a.x_out != nullptr, reinterpret_cast<T*>(a.h) + (size_t)row * pad8(a.W));
+}
+
+int launch_norm_rows(const NormStep& a, int kind, int rows, cudaStream_t st) {
+    if (rows <= 0) return JB_OK;
+    if (!a.h || !a.next_w || !a.next_b || (!a.tokens && (!a.x || (!a.y && !a.y_exp) || !a.post_w || !a.post_b))) return set_error(JB_ERR_PTR, "norm rows: null pointer");
+    const size_t smem = (size_t)pad8(a.W) * sizeof(float);
+    if (a.W <= 0 || smem > 200 * 1024) return set_error(JB_ERR_LIMIT, "norm rows: width %d", a.W);
+    if (smem > 48 * 1024) {
+        JB_CUDA(cudaFuncSetAttribute(norm_rows_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        JB_CUDA(cudaFuncSetAttribute(norm_rows_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    }
+    if (kind == EK_BF16) JB_CUDA(launch_k(norm_rows_kernel<__nv_bfloat16>, dim3(rows), dim3(NR_THREADS), smem, st, pdl_enabled(), a));
+    else                 JB_CUDA(launch_k(norm_rows_kernel<float>, dim3(rows), dim3(NR_THREADS), smem, st, pdl_enabled(), a));
+    count_launch();
+    return JB_OK;
+}
+
+}  // namespace jb

@@ -1,0 +1,127 @@
+// layernorm.cuh — the residual step of layer-list models: one row of
+//     x' = embed[token]                      (start of the stack)
+//     x' = x + mult * LN(y; post)            (exit of a sublayer, normed before it is added)
+//     h  = LN(x'; next)                      (entry of the next sublayer)
+// with LN(v; w, b) = (v - mean) / sqrt(var + eps) * w + b, var the mean of the squared deviations.  All of it in fp32; h is
+// rounded to the activation type.  The same device function serves the row kernel of the prompt path (layernorm.cu) and
+// the prologue of the decode products (dense_gemv.cu), so both give the same bits.
+#pragma once
+#include "common.cuh"
+#include <cuda_bf16.h>
+
+namespace jb {
+
+constexpr int EK_F16 = 0, EK_INT8 = 1, EK_BF16 = 2, EK_F32 = 3;      // element kinds of caches and activations
+inline int elem_bytes(int kind) { return kind == EK_F32 ? 4 : kind == EK_INT8 ? 1 : 2; }
+__host__ __device__ inline int pad8(int n) { return (n + 7) & ~7; }
+
+struct NormStep {
+    const float* x = nullptr; float* x_out = nullptr;      // residual rows, fp32, stride pad8(W); x_out may be null
+    const int* tokens = nullptr; const void* embed = nullptr;   // start of the stack: embedding rows, stride pad8(W)
+    const float* y = nullptr;                              // sublayer output, fp32, stride pad8(W)
+    // or the weighted sum of expert outputs: y = sum_k wts[row][k] * y_exp[slots[row][k]], k < top
+    const void* y_exp = nullptr; const int* slots = nullptr; const float* wts = nullptr; int top = 0;
+    const float* post_w = nullptr; const float* post_b = nullptr;
+    float mult = 1.f;
+    const float* next_w = nullptr; const float* next_b = nullptr;   // norm vectors: pad8(W) floats, zero beyond W
+    void* h = nullptr;                                     // normed rows, activation type, stride pad8(W)
+    const int* row_index = nullptr;                        // optional: row i works on source row row_index[i]
+    int W = 0; float eps = 0.f;
+};
+// kind: EK_BF16 or EK_F32 (embedding, expert outputs and h)
+int launch_norm_rows(const NormStep& a, int kind, int rows, cudaStream_t st);
+
+#ifdef __CUDACC__
+__device__ __forceinline__ float to_f32(float v) { return v; }
+__device__ __forceinline__ float to_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
+template <typename T> __device__ __forceinline__ T from_f32(float v);
+template <> __device__ __forceinline__ float from_f32<float>(float v) { return v; }
+template <> __device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
+__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load4(const __nv_bfloat16* p) {
+    const uint2 w = *reinterpret_cast<const uint2*>(p);
+    return make_float4(__uint_as_float(w.x << 16), __uint_as_float(w.x & 0xFFFF0000u), __uint_as_float(w.y << 16), __uint_as_float(w.y & 0xFFFF0000u));
+}
+__device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+}
+
+// sum over the CTA, the same value on every thread; red: THREADS / 32 floats
+template <int THREADS>
+__device__ __forceinline__ float block_sum(float v, float* red) {
+    v = warp_sum(v);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+    __syncthreads();
+    float s = 0.f;
+    #pragma unroll
+    for (int i = 0; i < THREADS / 32; ++i) s += red[i];
+    __syncthreads();
+    return s;
+}
+// mean and 1/sqrt(var + eps) of buf[0..W)
+template <int THREADS>
+__device__ __forceinline__ void ln_stats(const float* buf, int W, float eps, float* red, float& mean, float& rstd) {
+    const int n4 = pad8(W) / 4;
+    float s = 0.f;
+    for (int i = threadIdx.x; i < n4; i += THREADS) { const float4 v = load4(buf + 4 * i); s += (v.x + v.y) + (v.z + v.w); }   // zero beyond W
+    mean = block_sum<THREADS>(s, red) / (float)W;
+    float q = 0.f;
+    for (int i = threadIdx.x; i < n4; i += THREADS) {
+        const float4 v = load4(buf + 4 * i);
+        const float d[4] = {v.x - mean, v.y - mean, v.z - mean, v.w - mean};
+        #pragma unroll
+        for (int e = 0; e < 4; ++e) if (4 * i + e < W) q = fmaf(d[e], d[e], q);
+    }
+    rstd = 1.0f / sqrtf(block_sum<THREADS>(q, red) / (float)W + eps);
+}
+// One row by the whole CTA.  buf: pad8(W) floats of shared memory (each thread touches only its own elements of it);
+// red: THREADS / 32 floats; h_out: where the normed row goes (shared or global).
+template <typename T, int THREADS>
+__device__ __forceinline__ void norm_step_row(const NormStep& a, int row, float* buf, float* red, bool write_x, T* h_out) {
+    const int ld = pad8(a.W), n4 = ld / 4, src = a.row_index ? a.row_index[row] : row;
+    const size_t off = (size_t)src * ld;
+    if (a.tokens) {
+        const T* e = reinterpret_cast<const T*>(a.embed) + (size_t)a.tokens[src] * ld;
+        for (int i = threadIdx.x; i < n4; i += THREADS) {
+            const float4 v = load4(e + 4 * i);
+            store4(buf + 4 * i, v);
+            if (write_x) store4(a.x_out + (size_t)row * ld + 4 * i, v);
+        }
+    } else {
+        if (a.y_exp) {
+            for (int i = threadIdx.x; i < n4; i += THREADS) {
+                float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+                for (int k = 0; k < a.top; ++k) {
+                    const float w = a.wts[(size_t)src * a.top + k];
+                    const float4 v = load4(reinterpret_cast<const T*>(a.y_exp) + (size_t)a.slots[(size_t)src * a.top + k] * ld + 4 * i);
+                    s.x = fmaf(w, v.x, s.x); s.y = fmaf(w, v.y, s.y); s.z = fmaf(w, v.z, s.z); s.w = fmaf(w, v.w, s.w);
+                }
+                store4(buf + 4 * i, s);
+            }
+        } else {
+            for (int i = threadIdx.x; i < n4; i += THREADS) store4(buf + 4 * i, load4(a.y + off + 4 * i));
+        }
+        float mean, rstd;
+        ln_stats<THREADS>(buf, a.W, a.eps, red, mean, rstd);
+        for (int i = threadIdx.x; i < n4; i += THREADS) {
+            const float4 v = load4(buf + 4 * i), x = load4(a.x + off + 4 * i), w = load4(a.post_w + 4 * i), b = load4(a.post_b + 4 * i);
+            float4 r;
+            r.x = x.x + a.mult * ((v.x - mean) * rstd * w.x + b.x); r.y = x.y + a.mult * ((v.y - mean) * rstd * w.y + b.y);
+            r.z = x.z + a.mult * ((v.z - mean) * rstd * w.z + b.z); r.w = x.w + a.mult * ((v.w - mean) * rstd * w.w + b.w);
+            store4(buf + 4 * i, r);
+            if (write_x) store4(a.x_out + (size_t)row * ld + 4 * i, r);
+        }
+    }
+    float mean, rstd;
+    ln_stats<THREADS>(buf, a.W, a.eps, red, mean, rstd);
+    for (int i = threadIdx.x; i < n4; i += THREADS) {
+        const float4 v = load4(buf + 4 * i), w = load4(a.next_w + 4 * i), b = load4(a.next_b + 4 * i);
+        store4(h_out + 4 * i, make_float4((v.x - mean) * rstd * w.x + b.x, (v.y - mean) * rstd * w.y + b.y, (v.z - mean) * rstd * w.z + b.z,
+                                          (v.w - mean) * rstd * w.w + b.w));
+    }
+}
+#endif
+
+}  // namespace jb

@@ -28,7 +28,7 @@
 // Every mbarrier wait is bounded; a wait that runs out sets the device status word, the kernel still frees
 // its tensor memory and returns.
 #include "mmq.cuh"
-#include <cuda.h>
+#include "tc.cuh"
 #include <type_traits>
 #include <cstdlib>
 
@@ -41,7 +41,6 @@ constexpr int TC_STAGE_BYTES = TC_A_BYTES + TC_B_BYTES;
 constexpr int TC_SMEM = TC_STAGES * TC_STAGE_BYTES + 1024;    // + alignment slack
 constexpr int TC_PRODUCERS = 256;      // two dequantising threads per weight row
 constexpr int TC_THREADS = 64 + TC_PRODUCERS + 128;   // TMA warp, MMA warp, 8 dequantising warps, 4 draining warps
-constexpr uint32_t TC_WAIT_LIMIT = 1u << 24;
 
 struct TcArgs {
     __half* y; const uint8_t* W; int type; int M, N, K;
@@ -51,59 +50,6 @@ struct TcArgs {
     int n_full, ksplit;       // output tiles [0, n_full) are computed whole; each later one ("tail" tile) as `ksplit` K ranges whose
     float* part;              // fp32 partials [ksplit][tail tile][token of the tile][128 rows] a second kernel sums
 };
-
-__device__ __forceinline__ void tma_load_2d(void* dst, const CUtensorMap* map, int x, int y, uint64_t* bar) {
-    asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];"
-                 ::"r"(smem_u32(dst)), "l"(map), "r"(x), "r"(y), "r"(smem_u32(bar)) : "memory");
-}
-// Bounded wait without a sleep between polls: in this kernel every wait sits on the critical path between the
-// tensor pipe and the warps that feed it, and a sleeping warp wakes up far later than the barrier flips.
-__device__ __forceinline__ bool tc_wait(uint64_t* bar, uint32_t parity) {
-    const uint32_t addr = smem_u32(bar);
-    unsigned long long t0 = 0;
-    for (uint32_t i = 0; i < TC_WAIT_LIMIT; ++i) {
-        uint32_t ok;
-#ifdef JB_TC_SPIN
-        asm volatile("{\n .reg .pred p;\n mbarrier.test_wait.parity.shared::cta.b64 p, [%1], %2;\n selp.u32 %0, 1, 0, p;\n}"
-                     : "=r"(ok) : "r"(addr), "r"(parity) : "memory");
-#else
-        asm volatile("{\n .reg .pred p;\n mbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n selp.u32 %0, 1, 0, p;\n}"
-                     : "=r"(ok) : "r"(addr), "r"(parity) : "memory");
-#endif
-        if (ok) return true;
-        if ((i & 1023u) == 1023u) {           // a poll may block for a hardware-defined interval: bound the wait in time as well
-            const unsigned long long t = global_ns();
-            if (!t0) t0 = t; else if (t - t0 > 2000000000ull) return false;
-        }
-    }
-    return false;
-}
-__device__ __forceinline__ void tc_fail(volatile int* fail, int* status) { *fail = 1; atomicExch(status, JB_ERR_TIMEOUT); }
-__device__ __forceinline__ void tc_fence_before() { asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory"); }
-__device__ __forceinline__ void tc_fence_after()  { asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory"); }
-__device__ __forceinline__ void tc_commit(uint64_t* bar) {
-    asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(smem_u32(bar)) : "memory");
-}
-__device__ __forceinline__ void tc_mma_f16(uint32_t d_tmem, uint64_t a_desc, uint64_t b_desc, uint32_t idesc, uint32_t accumulate) {
-    asm volatile(
-        "{\n\t.reg .pred p;\n\tsetp.ne.b32 p, %4, 0;\n\t"
-        "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}\n"
-        ::"r"(d_tmem), "l"(a_desc), "l"(b_desc), "r"(idesc), "r"(accumulate) : "memory");
-}
-// K-major operand tile, 128-byte rows, 128-byte swizzle, 8-row atoms 1024 bytes apart
-__device__ __forceinline__ uint64_t tc_smem_desc(uint32_t saddr) {
-    return (uint64_t)((saddr >> 4) & 0x3FFFu) | (1ull << 16) | (64ull << 32) | (1ull << 46) | (2ull << 61);
-}
-__device__ __forceinline__ void tc_ld32(uint32_t taddr, uint32_t (&r)[32]) {
-    asm volatile("tcgen05.ld.sync.aligned.32x32b.x32.b32 "
-                 "{%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31}, [%32];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]), "=r"(r[9]),
-                   "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]), "=r"(r[16]), "=r"(r[17]), "=r"(r[18]),
-                   "=r"(r[19]), "=r"(r[20]), "=r"(r[21]), "=r"(r[22]), "=r"(r[23]), "=r"(r[24]), "=r"(r[25]), "=r"(r[26]), "=r"(r[27]),
-                   "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
-                 : "r"(taddr));
-    asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-}
 
 // 16 bytes = 8 fp16 weights of row `rl` written at K-chunk `c` (0..7) of a swizzled 128-byte row
 __device__ __forceinline__ void tc_store_chunk(uint8_t* a_tile, int rl, int c, uint4 v) {
@@ -574,25 +520,6 @@ __global__ void mmq_tc_reduce_kernel(__half* y, __half* y2, const float* part, i
         const float v[4] = {sum.x, sum.y, sum.z, sum.w};
         for (int i = 0; i < 4 && row + i < M; ++i) dst[i] = __float2half_rn(v[i]);
     }
-}
-
-typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
-                                  const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
-                                  CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-
-static EncodeTiledFn encode_tiled_fn() {
-    static EncodeTiledFn fn = nullptr;
-    static bool tried = false;
-    if (!tried) {
-        tried = true;
-        void* p = nullptr;
-        cudaDriverEntryPointQueryResult qr;
-        if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &p, cudaEnableDefault, &qr) == cudaSuccess && qr == cudaDriverEntryPointSuccess)
-            fn = (EncodeTiledFn)p;
-        else
-            cudaGetLastError();
-    }
-    return fn;
 }
 
 // Token-tile width, the number of whole output tiles and the K ranges of each remaining ("tail") tile, chosen together.

@@ -124,6 +124,35 @@ float* KVCachePool::kv_scale_ptr(int layer, int pos, bool is_value) {
     return kv_scales_ + (int64_t)layer * 2 * region + (is_value ? region : 0) + (int64_t)pos * cfg_.n_kv_heads;
 }
 
+bool LayeredKVCache::init(int n_layers, const int* k_width, const int* v_width, const int* source, int max_context, int elem_bytes) {
+    destroy();
+    if (n_layers <= 0 || max_context <= 0 || elem_bytes <= 0) return false;
+    slabs_ = new (std::nothrow) Slab[n_layers];
+    if (!slabs_) return false;
+    n_layers_ = n_layers; max_context_ = max_context; elem_ = elem_bytes;
+    auto slab = [&](int width) { return ((int64_t)max_context * width * elem_bytes + 255) & ~255LL; };
+    int64_t at = 0;
+    for (int l = 0; l < n_layers; ++l) {
+        const int s = source[l];
+        if (s < 0 || s > l || (s < l && source[s] != s)) { destroy(); return false; }
+        if (s < l) { slabs_[l] = slabs_[s]; continue; }
+        slabs_[l].k_width = k_width[l]; slabs_[l].v_width = v_width[l];
+        slabs_[l].k_off = at; at += slab(k_width[l]);
+        slabs_[l].v_off = at; at += slab(v_width[l]);
+    }
+    bytes_ = at;
+    if (cudaMalloc(&base_, (size_t)at) != cudaSuccess) { cudaGetLastError(); base_ = nullptr; destroy(); return false; }
+    if (cudaMemset(base_, 0, (size_t)at) != cudaSuccess) { cudaGetLastError(); destroy(); return false; }
+    return true;
+}
+void LayeredKVCache::destroy() {
+    if (base_) cudaFree(base_);
+    delete[] slabs_;
+    base_ = nullptr; slabs_ = nullptr; n_layers_ = 0; bytes_ = 0;
+}
+void* LayeredKVCache::key_ptr(int layer, int pos) const { const Slab& s = slabs_[layer]; return (char*)base_ + s.k_off + (int64_t)pos * s.k_width * elem_; }
+void* LayeredKVCache::val_ptr(int layer, int pos) const { const Slab& s = slabs_[layer]; return (char*)base_ + s.v_off + (int64_t)pos * s.v_width * elem_; }
+
 bool ScratchPool::init(int64_t size_bytes) {
     base_ = nullptr; capacity_ = offset_ = 0;
     if (size_bytes <= 0 || cudaMalloc(&base_, (size_t)size_bytes) != cudaSuccess) {

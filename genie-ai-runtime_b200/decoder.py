@@ -1,5 +1,6 @@
-"""Decoder session over the C ABI (jllm_b200_decoder_*): the reference engine's per-token kernel
-sequence (src/engine/decode.cu:1169-1246, :2101-2194) with greedy sampling on the device."""
+"""Decoder sessions over the C ABI (jllm_b200_decoder_*) with greedy sampling on the device.  Session holds what every model
+family shares; Decoder is the K-quant family (the reference engine's per-token kernel sequence,
+src/engine/decode.cu:1169-1246, :2101-2194), LayeredDecoder (layered.py) the models described layer by layer."""
 from __future__ import annotations
 
 import ctypes as C
@@ -23,39 +24,15 @@ class ModelDesc(C.Structure):
                 ("output_norm", C.c_void_p), ("layers", C.POINTER(LayerDesc))]
 
 
-lib.jllm_b200_decoder_create.restype = C.c_void_p
 lib.jllm_b200_decoder_logits.restype = C.c_void_p
 
 FUSED, GRAPH, PREFILL = 1, 2, 16          # PREFILL: generate() runs the prompt through the batched prefill path
 
 
-class Decoder:
-    """`weights` is a dict shaped like oracle.gen_model(): per-layer (uint8 block image, ggml type) pairs
-    and float32 norm vectors, given as torch CUDA tensors (see `upload`)."""
+class Session:
+    """One request stream of a model: subclasses create the handle `_h` and set `vocab` and `max_context`."""
 
-    def __init__(self, cfg, weights, max_context, flags=FUSED | GRAPH):
-        self._keep = weights
-        L = cfg["n_layers"]
-        self._layers = (LayerDesc * L)()
-        names = dict(wq="wq", wk="wk", wv="wv", wo="wo", w_gate="gate", w_up="up", w_down="down")
-        for i, lw in enumerate(weights["layers"]):
-            for f, k in names.items():
-                setattr(self._layers[i], f, lw[k][0].data_ptr())
-                setattr(self._layers[i], "type_" + f, lw[k][1])
-            for k in ("rms_attn", "rms_ffn", "q_norm", "k_norm"):
-                setattr(self._layers[i], k, lw[k].data_ptr() if lw.get(k) is not None else None)
-        m = ModelDesc()
-        m.n_layers, m.hidden_dim, m.n_heads, m.n_kv_heads = L, cfg["hidden"], cfg["n_heads"], cfg["n_kv_heads"]
-        m.head_dim, m.intermediate_dim, m.vocab_size, m.max_context = cfg["head_dim"], cfg["ffn"], cfg["vocab"], max_context
-        m.rope_theta, m.rms_eps, m.rope_neox = cfg["rope_theta"], cfg["eps"], 1
-        m.tok_embd, m.embd_type = weights["tok_embd"][0].data_ptr(), weights["tok_embd"][1]
-        m.output, m.output_type = weights["output"][0].data_ptr(), weights["output"][1]
-        m.output_norm = weights["out_norm"].data_ptr()
-        m.layers = self._layers
-        self.cfg, self.max_context = cfg, max_context
-        self._h = lib.jllm_b200_decoder_create(C.byref(m), C.c_int(flags))
-        if not self._h:
-            raise JllmError(-1, last_error())
+    _h = None
 
     def close(self):
         if self._h:
@@ -85,13 +62,23 @@ class Decoder:
             check(lib.jllm_b200_decoder_set_prefill_chunk(C.c_void_p(self._h), C.c_int(chunk)))
         check(lib.jllm_b200_decoder_prefill(C.c_void_p(self._h), t.ctypes.data_as(C.c_void_p), C.c_int(t.size), C.c_int(start_pos), _stream(stream)))
 
+    def feed(self, tokens, start_pos=0, want=(), stream=None):
+        """Runs host tokens at positions start_pos .. (one token: the decode step; more: the chunk path) and returns the
+        logits at the wanted places among them, float32 [len(want), vocab].  Nothing is sampled."""
+        t = np.ascontiguousarray(tokens, np.int32)
+        w = np.ascontiguousarray(want, np.int32)
+        out = np.empty((w.size, self.vocab), np.float32)
+        check(lib.jllm_b200_decoder_feed(C.c_void_p(self._h), t.ctypes.data_as(C.c_void_p), C.c_int(t.size), C.c_int(start_pos),
+                                         w.ctypes.data_as(C.c_void_p), C.c_int(w.size), out.ctypes.data_as(C.c_void_p), _stream(stream)))
+        return out
+
     def last_token(self, stream=None):
         return int(lib.jllm_b200_decoder_last_token(C.c_void_p(self._h), _stream(stream)))
 
     def logits(self):
         import torch
         ptr = lib.jllm_b200_decoder_logits(C.c_void_p(self._h))
-        out = torch.empty(self.cfg["vocab"], dtype=torch.float32, device="cuda")
+        out = torch.empty(self.vocab, dtype=torch.float32, device="cuda")
         torch.cuda.synchronize()
         C.CDLL("libcudart.so").cudaMemcpy(C.c_void_p(out.data_ptr()), C.c_void_p(ptr), C.c_size_t(out.numel() * 4), 3)
         return out
@@ -112,6 +99,36 @@ class Decoder:
         out = np.zeros(max(n, 1), np.int32)
         cnt = int(lib.jllm_b200_decoder_recorded_tokens(C.c_void_p(self._h), C.c_int(first), C.c_int(n), out.ctypes.data_as(C.c_void_p), _stream(stream)))
         return cnt, out[:max(0, min(n, cnt - first))]
+
+
+class Decoder(Session):
+    """`weights` is a dict shaped like oracle.gen_model(): per-layer (uint8 block image, ggml type) pairs
+    and float32 norm vectors, given as torch CUDA tensors (see `upload`)."""
+
+    def __init__(self, cfg, weights, max_context, flags=FUSED | GRAPH):
+        self._keep = weights
+        L = cfg["n_layers"]
+        self._layers = (LayerDesc * L)()
+        names = dict(wq="wq", wk="wk", wv="wv", wo="wo", w_gate="gate", w_up="up", w_down="down")
+        for i, lw in enumerate(weights["layers"]):
+            for f, k in names.items():
+                setattr(self._layers[i], f, lw[k][0].data_ptr())
+                setattr(self._layers[i], "type_" + f, lw[k][1])
+            for k in ("rms_attn", "rms_ffn", "q_norm", "k_norm"):
+                setattr(self._layers[i], k, lw[k].data_ptr() if lw.get(k) is not None else None)
+        m = ModelDesc()
+        m.n_layers, m.hidden_dim, m.n_heads, m.n_kv_heads = L, cfg["hidden"], cfg["n_heads"], cfg["n_kv_heads"]
+        m.head_dim, m.intermediate_dim, m.vocab_size, m.max_context = cfg["head_dim"], cfg["ffn"], cfg["vocab"], max_context
+        m.rope_theta, m.rms_eps, m.rope_neox = cfg["rope_theta"], cfg["eps"], 1
+        m.tok_embd, m.embd_type = weights["tok_embd"][0].data_ptr(), weights["tok_embd"][1]
+        m.output, m.output_type = weights["output"][0].data_ptr(), weights["output"][1]
+        m.output_norm = weights["out_norm"].data_ptr()
+        m.layers = self._layers
+        self.cfg, self.max_context, self.vocab = cfg, max_context, cfg["vocab"]
+        lib.jllm_b200_decoder_create.restype = C.c_void_p
+        self._h = lib.jllm_b200_decoder_create(C.byref(m), C.c_int(flags))
+        if not self._h:
+            raise JllmError(-1, last_error())
 
 
 class BatchDecoder:

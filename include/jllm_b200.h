@@ -278,6 +278,42 @@ int    jllm_b200_decoder_recorded_tokens(jllm_b200_decoder* d, int first, int n,
  * 7 layer-0 K cache, 8 layer-0 K scales. */
 const void* jllm_b200_decoder_buffer(jllm_b200_decoder* d, int which);
 
+/* ── decoder session of a model described layer by layer (extension) ─────────────────────────────────────
+ * The same session (every jllm_b200_decoder_* function below and above) over layers that may differ from one another:
+ *     x = embed[token];   per layer  x += mult * LN(mixer(LN(x; norm1)); norm1b),  x += mult * LN(mlp(LN(x; norm2)); norm2b)
+ *     logits = softcap(embed . LN(x; final))
+ * with an fp32 residual.  Mixer: causal grouped-query attention without rotation, a query temperature, a softmax sink per
+ * head, optionally over the keys and values of an earlier layer.  MLP: none, or a mixture of SwiGLU experts with sigmoid
+ * routing.  dtype: 2 = bf16 weights, activations and cache (tensor cores, fp32 accumulation; norms, routing, softmax and
+ * residual in fp32), 3 = everything in fp32.
+ * Weights are device matrices of dtype, row-major [out][in], rows padded to a multiple of 8 elements with zeros; norm
+ * vectors are fp32, padded to a multiple of 8 with zeros; biases likewise. */
+typedef struct {
+    /* mixer: attention */
+    int n_heads, n_kv_heads, head_dim, v_dim;
+    int kv_from;                              /* earlier layer whose keys and values are used, or -1 */
+    float scale, q_temp_coef; double q_temp_every;   /* q_temp_every <= 0: no temperature */
+    const void *w_qkv;                        /* q rows, then k rows, then v rows (q rows only with kv_from) */
+    const void *w_o;                          /* [width][n_heads * v_dim] */
+    const float *sink;                        /* [n_heads] or null */
+    const float *norm1_w, *norm1_b, *norm1b_w, *norm1b_b;
+    /* mlp: mixture of experts, n_experts = 0 for none */
+    int n_experts, top, n_groups, keep_groups, expert_dim;      /* n_groups = 1: no groups */
+    const void *w_router;                     /* [n_experts][width] */
+    const float *correction;                  /* [n_experts] or null */
+    const void *w_gate, *w_up, *w_down;       /* [n_experts][expert_dim][width] twice, [n_experts][width][expert_dim] */
+    const float *norm2_w, *norm2_b, *norm2b_w, *norm2b_b;
+} jllm_b200_layer_spec;
+typedef struct {
+    int n_layers, width, vocab_size, max_context, dtype;
+    float eps, residual_mult, logit_softcap;  /* logit_softcap <= 0: none */
+    const void *embed;                        /* [vocab_size][width], also the output matrix */
+    const float *final_w, *final_b;
+    const jllm_b200_layer_spec *layers;
+} jllm_b200_layered_desc;
+/* flags: bit 1 = CUDA graph per step, bit 4 = generate() runs the prompt through the chunk path */
+jllm_b200_decoder* jllm_b200_decoder_create_layered(const jllm_b200_layered_desc* model, int flags);
+
 /* ── tensor-parallel decoder session (extension; the reference is single-GPU) ───────────────────────────
  * One process per GPU.  Rank r of `world` (2, 4 or 8) owns rows [r*M/world, (r+1)*M/world) of every weight matrix
  * (a contiguous byte range of the GGUF image) and the KV heads that go with its query heads.  `model` carries the

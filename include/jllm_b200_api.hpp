@@ -139,4 +139,24 @@ private:
     int64_t offset_ = 0;
 };
 
+// Extension: cache slab of models whose layers differ.  Keys and values of a layer have their own widths (elements per
+// position), and a layer may read the keys and values of an earlier one (source[l] != l) and then holds none itself.
+// Per owning layer: keys of every position, then values of every position; slabs start 256-byte aligned.
+class LayeredKVCache {
+public:
+    bool  init(int n_layers, const int* k_width, const int* v_width, const int* source, int max_context, int elem_bytes);
+    void  destroy();
+    void* key_ptr(int layer, int pos) const;
+    void* val_ptr(int layer, int pos) const;
+    int64_t capacity_bytes() const { return bytes_; }
+    int  max_context() const { return max_context_; }
+
+private:
+    struct Slab { int64_t k_off, v_off; int k_width, v_width; };
+    void*   base_ = nullptr;
+    Slab*   slabs_ = nullptr;          // per layer; a sharing layer repeats its source's
+    int     n_layers_ = 0, max_context_ = 0, elem_ = 0;
+    int64_t bytes_ = 0;
+};
+
 }  // namespace jllm
