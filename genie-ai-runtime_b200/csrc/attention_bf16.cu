@@ -49,7 +49,7 @@ template <int D> __device__ __forceinline__ uint32_t fa_off(int r, int c) { retu
 
 // One 16-row step over NK keys (a multiple of 16) whose K / V tiles sit in shared memory: S = Q K^T, online softmax in base
 // 2, O += P V.  qf(ks) gives the A fragment of k-step ks.  live(row_half, key) masks; fsc[2] = score factors of the two rows.
-template <int D, int NK, class QF, class Live>
+template <int D, int NK, bool FULL, class QF, class Live>
 __device__ __forceinline__ void fa_step(float (&o)[D / 8][4], float (&m)[2], float (&l)[2], const float (&fsc)[2], uint32_t ks_addr, uint32_t vs_addr,
                                         int dim, int vdim, bool masked, QF qf, Live live) {
     const int lane = threadIdx.x & 31, lr = lane & 7, lm = lane >> 3;
@@ -58,7 +58,7 @@ __device__ __forceinline__ void fa_step(float (&o)[D / 8][4], float (&m)[2], flo
     for (int i = 0; i < NK / 8; ++i) { s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f; }
     #pragma unroll
     for (int ks = 0; ks < D / 16; ++ks) {
-        if (ks * 16 < dim) {
+        if (FULL || ks * 16 < dim) {
             uint32_t a[4];
             qf(ks, a);
             #pragma unroll
@@ -108,7 +108,7 @@ __device__ __forceinline__ void fa_step(float (&o)[D / 8][4], float (&m)[2], flo
                                fa_pack(s[2 * kk + 1][0], s[2 * kk + 1][1]), fa_pack(s[2 * kk + 1][2], s[2 * kk + 1][3])};
         #pragma unroll
         for (int dt = 0; dt < D / 16; ++dt) {
-            if (dt * 16 < vdim) {                            // transposed matrices: keys 0-7 | 8-15, then the next 8 dims
+            if (FULL || dt * 16 < vdim) {                            // transposed matrices: keys 0-7 | 8-15, then the next 8 dims
                 uint32_t b[4];
                 fa_ldsm_t(b, vs_addr + fa_off<D>(kk * 16 + (lm & 1) * 8 + lr, dt * 2 + (lm >> 1)));
                 fa_mma(o[2 * dt], a, b[0], b[1]);
@@ -118,15 +118,27 @@ __device__ __forceinline__ void fa_step(float (&o)[D / 8][4], float (&m)[2], flo
     }
 }
 
-// rows [row0, row0 + n) of a cache matrix into a swizzled tile; chunks up to the 16-element round-up of `width`, zero beyond
-// the real width and beyond row `end`
-template <int D>
-__device__ __forceinline__ void fa_load_rows(uint32_t tile, const __nv_bfloat16* base, int ld, int width, int row0, int n, int end, int tid, int threads) {
-    const int ch = ((width + 15) >> 4) * 2, real = width >> 3;
-    for (int i = tid; i < n * ch; i += threads) {
-        const int r = i / ch, c = i - r * ch;
-        const bool in = row0 + r < end && c < real;
-        fa_cp16(tile + fa_off<D>(r, c), in ? base + (size_t)(row0 + r) * ld + c * 8 : base, in);
+// rows [row0, row0 + N) of a cache matrix into a swizzled tile; chunks up to the 16-element round-up of `width`, zero beyond
+// the real width and beyond row `end`.  FULL: width = D, so a lane keeps its chunk and steps over rows.
+template <int D, bool FULL, int N, int THREADS>
+__device__ __forceinline__ void fa_load_rows(uint32_t tile, const __nv_bfloat16* base, int ld, int width, int row0, int end, int tid) {
+    if constexpr (FULL && THREADS % (D / 8) == 0) {
+        constexpr int STEP = THREADS / (D / 8);
+        const int c = tid % (D / 8), r0 = tid / (D / 8);
+        const __nv_bfloat16* p = base + (size_t)(row0 + r0) * ld + c * 8;
+        #pragma unroll
+        for (int i = 0; i < N / STEP; ++i) {
+            const int r = r0 + i * STEP;
+            const bool in = row0 + r < end;
+            fa_cp16(tile + fa_off<D>(r, c), in ? p + (size_t)(i * STEP) * ld : base, in);
+        }
+    } else {
+        const int ch = ((width + 15) >> 4) * 2, real = width >> 3;
+        for (int i = tid; i < N * ch; i += THREADS) {
+            const int r = i / ch, c = i - r * ch;
+            const bool in = row0 + r < end && c < real;
+            fa_cp16(tile + fa_off<D>(r, c), in ? base + (size_t)(row0 + r) * ld + c * 8 : base, in);
+        }
     }
 }
 
@@ -136,7 +148,7 @@ template <int D> constexpr bool fp_q_in_regs() { return D <= 128; }
 // two stages of K and V; the query tile shares the second K stage when its fragments live in registers
 template <int D> constexpr int fp_smem() { return (4 + (fp_q_in_regs<D>() ? 0 : 1)) * FP_KEYS * D * 2; }
 
-template <int D>
+template <int D, bool FULL>
 __global__ void __launch_bounds__(FP_THREADS) attn_bf16_prefill_kernel(const FaArgs a) {
     pdl_wait();
     extern __shared__ __align__(128) unsigned char fp_sm[];
@@ -158,8 +170,8 @@ __global__ void __launch_bounds__(FP_THREADS) attn_bf16_prefill_kernel(const FaA
         }
         fa_commit();
     }
-    fa_load_rows<D>(sm, kb, a.ldk, a.dim, 0, FP_KEYS, n_keys, tid, FP_THREADS);
-    fa_load_rows<D>(sm + 2 * TB, vb, a.ldv, a.vdim, 0, FP_KEYS, n_keys, tid, FP_THREADS);
+    fa_load_rows<D, FULL, FP_KEYS, FP_THREADS>(sm, kb, a.ldk, a.dim, 0, n_keys, tid);
+    fa_load_rows<D, FULL, FP_KEYS, FP_THREADS>(sm + 2 * TB, vb, a.ldv, a.vdim, 0, n_keys, tid);
     fa_commit();
     uint32_t qreg[fp_q_in_regs<D>() ? D / 16 : 1][4];
     const uint32_t q_lane = (uint32_t)(warp * 16 + (lane & 15));
@@ -167,7 +179,7 @@ __global__ void __launch_bounds__(FP_THREADS) attn_bf16_prefill_kernel(const FaA
         fa_wait<1>();
         __syncthreads();
         #pragma unroll
-        for (int ks = 0; ks < D / 16; ++ks) if (ks * 16 < a.dim) fa_ldsm(qreg[fp_q_in_regs<D>() ? ks : 0], qst + fa_off<D>((int)q_lane, ks * 2 + (lane >> 4)));
+        for (int ks = 0; ks < D / 16; ++ks) if (FULL || ks * 16 < a.dim) fa_ldsm(qreg[fp_q_in_regs<D>() ? ks : 0], qst + fa_off<D>((int)q_lane, ks * 2 + (lane >> 4)));
         __syncthreads();                                   // the second K stage is free for keys
     }
     auto qf = [&](int ks, uint32_t (&f)[4]) {
@@ -190,15 +202,15 @@ __global__ void __launch_bounds__(FP_THREADS) attn_bf16_prefill_kernel(const FaA
     for (int t = 0; t < tiles; ++t) {
         const uint32_t b = t & 1;
         if (t + 1 < tiles) {
-            fa_load_rows<D>(sm + (b ^ 1) * TB, kb, a.ldk, a.dim, (t + 1) * FP_KEYS, FP_KEYS, n_keys, tid, FP_THREADS);
-            fa_load_rows<D>(sm + (2 + (b ^ 1)) * TB, vb, a.ldv, a.vdim, (t + 1) * FP_KEYS, FP_KEYS, n_keys, tid, FP_THREADS);
+            fa_load_rows<D, FULL, FP_KEYS, FP_THREADS>(sm + (b ^ 1) * TB, kb, a.ldk, a.dim, (t + 1) * FP_KEYS, n_keys, tid);
+            fa_load_rows<D, FULL, FP_KEYS, FP_THREADS>(sm + (2 + (b ^ 1)) * TB, vb, a.ldv, a.vdim, (t + 1) * FP_KEYS, n_keys, tid);
         }
         fa_commit();
         fa_wait<1>();
         __syncthreads();
         const int k0 = t * FP_KEYS;
         if (k0 <= warp_last)
-            fa_step<D, FP_KEYS>(o, m, l, fsc, sm + b * TB, sm + (2 + b) * TB, a.dim, a.vdim, k0 + FP_KEYS - 1 > warp_first, qf, [&](int h, int key) { return k0 + key <= pos[h]; });
+            fa_step<D, FP_KEYS, FULL>(o, m, l, fsc, sm + b * TB, sm + (2 + b) * TB, a.dim, a.vdim, k0 + FP_KEYS - 1 > warp_first, qf, [&](int h, int key) { return k0 + key <= pos[h]; });
         __syncthreads();
     }
     #pragma unroll
@@ -226,7 +238,7 @@ template <int D> constexpr int fd_smem() {
     return FD_WARPS * fd_stages<D>() * 2 * FD_KEYS * D * 2 > FD_WARPS * 16 * (D + 2) * 4 ? FD_WARPS * fd_stages<D>() * 2 * FD_KEYS * D * 2 : FD_WARPS * 16 * (D + 2) * 4;
 }
 
-template <int D>
+template <int D, bool FULL>
 __global__ void __launch_bounds__(FD_THREADS) attn_bf16_decode_kernel(const FaArgs a) {
     pdl_wait();
     extern __shared__ __align__(128) unsigned char fd_sm[];
@@ -259,8 +271,8 @@ __global__ void __launch_bounds__(FD_THREADS) attn_bf16_decode_kernel(const FaAr
     auto fetch = [&](int i) {
         const int k0 = k_lo + (warp + i * FD_WARPS) * FD_KEYS;
         const uint32_t st = ring + (uint32_t)(i % ST) * 2 * TB;
-        fa_load_rows<D>(st, kb, a.ldk, a.dim, k0, FD_KEYS, k_hi, lane, 32);
-        fa_load_rows<D>(st + TB, vb, a.ldv, a.vdim, k0, FD_KEYS, k_hi, lane, 32);
+        fa_load_rows<D, FULL, FD_KEYS, 32>(st, kb, a.ldk, a.dim, k0, k_hi, lane);
+        fa_load_rows<D, FULL, FD_KEYS, 32>(st + TB, vb, a.ldv, a.vdim, k0, k_hi, lane);
     };
     #pragma unroll
     for (int i = 0; i < ST - 1; ++i) { if (i < mine) fetch(i); fa_commit(); }
@@ -269,7 +281,7 @@ __global__ void __launch_bounds__(FD_THREADS) attn_bf16_decode_kernel(const FaAr
         __syncwarp();
         const int k0 = k_lo + (warp + i * FD_WARPS) * FD_KEYS;
         const uint32_t st = ring + (uint32_t)(i % ST) * 2 * TB;
-        fa_step<D, FD_KEYS>(o, m, l, fsc, st, st + TB, a.dim, a.vdim, k0 + FD_KEYS > k_hi,
+        fa_step<D, FD_KEYS, FULL>(o, m, l, fsc, st, st + TB, a.dim, a.vdim, k0 + FD_KEYS > k_hi,
                             [&](int ks, uint32_t (&fr)[4]) { for (int e = 0; e < 4; ++e) fr[e] = qreg[ks][e]; }, [&](int, int key) { return k0 + key < k_hi; });
         __syncwarp();
         if (i + ST - 1 < mine) fetch(i + ST - 1);
@@ -370,22 +382,27 @@ int attn_bf16_splits(int seq_len, int n_heads, int n_kv) {
     return n;
 }
 
-template <int D>
-static int fa_launch(const FaArgs& a, bool prefill, cudaStream_t st) {
+template <int D, bool FULL>
+static int fa_launch_t(const FaArgs& a, bool prefill, cudaStream_t st) {
     static bool attr = false;
     if (!attr) {
-        JB_CUDA(cudaFuncSetAttribute(attn_bf16_prefill_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, fp_smem<D>()));
-        JB_CUDA(cudaFuncSetAttribute(attn_bf16_decode_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, fd_smem<D>()));
+        JB_CUDA(cudaFuncSetAttribute(attn_bf16_prefill_kernel<D, FULL>, cudaFuncAttributeMaxDynamicSharedMemorySize, fp_smem<D>()));
+        JB_CUDA(cudaFuncSetAttribute(attn_bf16_decode_kernel<D, FULL>, cudaFuncAttributeMaxDynamicSharedMemorySize, fd_smem<D>()));
         attr = true;
     }
     if (prefill) {
         const long long rows = (long long)a.n_tokens * a.R;
-        JB_CUDA(launch_k(attn_bf16_prefill_kernel<D>, dim3((unsigned)((rows + FP_ROWS - 1) / FP_ROWS), a.n_kv), dim3(FP_THREADS), fp_smem<D>(), st, pdl_enabled(), a));
+        JB_CUDA(launch_k(attn_bf16_prefill_kernel<D, FULL>, dim3((unsigned)((rows + FP_ROWS - 1) / FP_ROWS), a.n_kv), dim3(FP_THREADS), fp_smem<D>(), st, pdl_enabled(), a));
     } else {
-        JB_CUDA(launch_k(attn_bf16_decode_kernel<D>, dim3(a.n_kv * a.row_blocks, a.n_splits), dim3(FD_THREADS), fd_smem<D>(), st, pdl_enabled(), a));
+        JB_CUDA(launch_k(attn_bf16_decode_kernel<D, FULL>, dim3(a.n_kv * a.row_blocks, a.n_splits), dim3(FD_THREADS), fd_smem<D>(), st, pdl_enabled(), a));
     }
     count_launch();
     return JB_OK;
+}
+
+template <int D>
+static int fa_launch(const FaArgs& a, bool prefill, cudaStream_t st) {
+    return a.dim == D && a.vdim == D ? fa_launch_t<D, true>(a, prefill, st) : fa_launch_t<D, false>(a, prefill, st);
 }
 
 int launch_attention_bf16(const AttnCall& c, cudaStream_t st) {

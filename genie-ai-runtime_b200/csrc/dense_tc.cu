@@ -75,13 +75,16 @@ __global__ void __launch_bounds__(DT_THREADS, 1) dense_tc_kernel(const __grid_co
     const uint32_t tmem = tmem_slot;
     const int n_work = t_first[a.n_groups];
     int grp = 0;
-    // work item w -> group, weight row tile, first token row (the groups are walked in order; within one, token tiles fastest)
+    // work item w -> weight row tile, token rows [n0, n_end) (the groups are walked in order; within one, token tiles fastest).
+    // A group's tokens are dealt evenly to as few tiles as n_tile allows, and the MMA of a tile is only as wide as its tokens.
     auto locate = [&](int w, int& mt, int& n0, int& n_end) {
         while (w >= t_first[grp + 1]) ++grp;
-        n_end = row_off[grp + 1];
-        const int tn = (n_end - row_off[grp] + a.n_tile - 1) / a.n_tile, i = w - t_first[grp];
+        const int lo = row_off[grp], count = row_off[grp + 1] - lo, i = w - t_first[grp];
+        const int tn = (count + a.n_tile - 1) / a.n_tile, width = ((count + tn - 1) / tn + 15) & ~15;
         mt = i / tn;
-        n0 = row_off[grp] + (i - mt * tn) * a.n_tile;
+        const int nt = i - mt * tn;
+        n0 = lo + min(nt * width, count);
+        n_end = lo + min((nt + 1) * width, count);
     };
 
     if (warp == 0) {
@@ -105,13 +108,16 @@ __global__ void __launch_bounds__(DT_THREADS, 1) dense_tc_kernel(const __grid_co
         }
     } else if (warp == 1) {
         if (lane == 0) {
-            // bf16 x bf16 -> fp32, both operands K-major, M = 128, N = n_tile
-            const uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(a.n_tile >> 3) << 17) | ((uint32_t)(DT_M >> 4) << 24);
+            // bf16 x bf16 -> fp32, both operands K-major, M = 128, N = the tile's tokens rounded up to 16
+            const uint32_t idesc0 = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(DT_M >> 4) << 24);
             const uint64_t ad0 = tc_smem_desc(smem_u32(smem)), bd0 = tc_smem_desc(smem_u32(smem + A_BYTES));
             uint32_t it = 0, j = 0;
             bool ok = true;
             for (int w = blockIdx.x; w < n_work && ok; w += gridDim.x, ++j) {
                 const uint32_t d = tmem + (j & 1) * 256u;
+                int mt, n0, n_end;
+                locate(w, mt, n0, n_end);
+                const uint32_t idesc = idesc0 | ((uint32_t)max(2, ((n_end - n0 + 15) >> 4) * 2) << 17);
                 if (!tc_wait(&acc_empty[j & 1], ((j >> 1) & 1) ^ 1)) { ok = false; break; }
                 tc_fence_after();
                 for (int t = 0; t < a.k_tiles; ++t, ++it) {
@@ -152,7 +158,7 @@ __global__ void __launch_bounds__(DT_THREADS, 1) dense_tc_kernel(const __grid_co
             const bool f32 = a.seg[s].f32 != 0;
             float* yf = reinterpret_cast<float*>(a.seg[s].y) + row;
             __nv_bfloat16* yb = reinterpret_cast<__nv_bfloat16*>(a.seg[s].y) + row;
-            const int cols = min(a.n_tile, n_end - n0);
+            const int cols = n_end - n0;
             const uint32_t t_acc = tmem + ((uint32_t)(q * 32) << 16) + acc * 256u;
             for (int cb = 0; cb < cols; cb += 32) {
                 uint32_t r[32];
@@ -189,15 +195,17 @@ __global__ void __launch_bounds__(DT_THREADS, 1) dense_tc_kernel(const __grid_co
     }
 }
 
-// Token-tile width: wide tiles use the tensor pipe best, but too few of them leave SMs idle for the last round.
+// Widest token tile: wide tiles use the tensor pipe best, but too few of them leave SMs idle in the last round.  A tile costs
+// about its width, with a floor (below it the weight tile's bandwidth sets the time).
 static int dt_pick(int tiles_m, int tokens_per_group, int groups, int max_tile, int sm) {
-    int best = 32;
+    int best = max_tile;
     double cost = 1e30;
-    for (int c = 32; c <= max_tile; c <<= 1) {
-        if (c > 32 && c / 2 >= tokens_per_group) break;
-        const long long tiles = (long long)groups * tiles_m * ((tokens_per_group + c - 1) / c);
-        const double t = (double)((tiles + sm - 1) / sm) * ((c < 128 ? 128 : c) / 256.0 + 0.02);
-        if (t <= cost) { cost = t; best = c; }
+    for (int c = 16; c <= max_tile; c += 16) {
+        if (c > 16 && c - 16 >= tokens_per_group) break;
+        const int tn = (tokens_per_group + c - 1) / c, width = ((tokens_per_group + tn - 1) / tn + 15) & ~15;
+        const long long tiles = (long long)groups * tiles_m * tn;
+        const double t = (double)((tiles + sm - 1) / sm) * ((width < 96 ? 96 : width) + 8);
+        if (t < cost) { cost = t; best = c; }
     }
     return best;
 }
@@ -214,7 +222,9 @@ int launch_dense_gemm_tc(const DenseGemm& a, cudaStream_t st) {
     p.nseg = a.nseg; p.M = a.M; p.N = a.N; p.n_groups = a.n_groups; p.softcap = a.softcap; p.off = a.off; p.status = c->d_status;
     p.k_tiles = (a.K + DT_K - 1) / DT_K;
     const int tiles_m = (a.M + DT_M - 1) / DT_M, per = (a.N + a.n_groups - 1) / a.n_groups;
-    p.n_tile = dt_pick(tiles_m, per, a.n_groups, a.swiglu ? 128 : 256, c->sm_count);
+    // groups: widest tile, the kernel narrows each to its group's tokens (a few groups hold more than the average)
+    p.n_tile = a.n_groups > 1 ? (per >= (a.swiglu ? 96 : 192) ? (a.swiglu ? 128 : 256) : ((per + per / 4 + 31) & ~15)) : dt_pick(tiles_m, per, 1, a.swiglu ? 128 : 256, c->sm_count);
+    if (p.n_tile > (a.swiglu ? 128 : 256)) p.n_tile = a.swiglu ? 128 : 256;
     CUtensorMap wm, um, xm;
     const long long ld = pad8(a.K);
     if (!encode_tile_map(&wm, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, a.W, (long long)a.n_groups * a.M, a.K, ld, DT_M) ||

@@ -205,6 +205,49 @@ def flash_attention_decode_noalloc(output, q, k_cache, v_cache, n_heads, n_kv_he
                                                        _stream(stream)))
 
 
+_KINDS = {"torch.bfloat16": 2, "torch.float32": 3}
+
+
+def _kind(t):
+    return i32(_KINDS[str(t.dtype)])
+
+
+def norm_step(h, x_out, next_w, next_b, eps, width, mult=1.0, x=None, y=None, tokens=None, embed=None, y_exp=None, slots=None, weights=None,
+              post_w=None, post_b=None, stream=None):
+    check(lib.jllm_b200_norm_step(_ptr(h), _ptr(x_out), _ptr(x), _ptr(y), _ptr(tokens), _ptr(embed), _ptr(y_exp), _ptr(slots), _ptr(weights),
+                                  i32(weights.shape[1] if weights is not None else 0), _ptr(post_w), _ptr(post_b), _ptr(next_w), _ptr(next_b),
+                                  f32(mult), f32(eps), i32(h.shape[0]), i32(width), _kind(h), _stream(stream)))
+
+
+def sink_attention(out, q, k, v, n_heads, n_kv_heads, head_dim, v_dim, scale, n_tokens=0, start=0, seq_len=0, sink=None, q_temp=(0.0, 0.0), n_splits=0,
+                   stream=None):
+    """n_tokens > 0: causal queries at start ..; n_tokens = 0: one query over seq_len keys."""
+    check(lib.jllm_b200_sink_attention(_ptr(out), _ptr(q), _ptr(k), _ptr(v), _kind(q), i32(n_heads), i32(n_kv_heads), i32(head_dim), i32(v_dim),
+                                       i32(n_tokens), i32(start), i32(seq_len), f32(scale), _ptr(sink), f32(q_temp[0]), C.c_double(q_temp[1]),
+                                       i32(n_splits), _stream(stream)))
+
+
+def moe_route(ids, weights, rank, counts, z, top, n_groups=1, keep_groups=1, correction=None, stream=None):
+    check(lib.jllm_b200_moe_route(_ptr(ids), _ptr(weights), _ptr(rank), _ptr(counts), _ptr(z), _ptr(correction), i32(z.shape[0]), i32(z.shape[1]),
+                                  i32(top), i32(n_groups), i32(keep_groups), _stream(stream)))
+
+
+def dense_matmul(y, W, x, M, N, K, W_up=None, group_offsets=None, n_groups=1, softcap=0.0, stream=None):
+    check(lib.jllm_b200_dense_matmul(_ptr(y), _ptr(W), _ptr(W_up), _ptr(x), _ptr(group_offsets), i32(n_groups), _kind(x),
+                                     i32(1 if str(y.dtype) == "torch.float32" else 0), i32(M), i32(N), i32(K), f32(softcap), _stream(stream)))
+
+
+def dense_matvec(y, W, x, M, K, softcap=0.0, stream=None):
+    check(lib.jllm_b200_dense_matvec(_ptr(y), _ptr(W), _ptr(x), _kind(x), i32(1 if str(y.dtype) == "torch.float32" else 0), i32(M), i32(K), f32(softcap),
+                                     _stream(stream)))
+
+
+def moe_matvec(y, act, ids, weights, W_gate, W_up, W_down, h, z, top, ff, width, n_groups=1, keep_groups=1, correction=None, stream=None):
+    check(lib.jllm_b200_moe_matvec(_ptr(y), _ptr(act), _ptr(ids), _ptr(weights), _ptr(W_gate), _ptr(W_up), _ptr(W_down), _ptr(h), _ptr(z),
+                                   _ptr(correction), _kind(h), i32(z.shape[-1]), i32(top), i32(n_groups), i32(keep_groups), i32(ff), i32(width),
+                                   _stream(stream)))
+
+
 class AttnPlan:
     """Ragged batched decode attention over a fixed set of INT8 caches (jllm_b200_attn_plan_*): the tensor maps of the
     caches are built once; `k_list` ... `vs_list` are sequences of torch CUDA tensors (one per sequence), every cache

@@ -314,6 +314,36 @@ typedef struct {
 /* flags: bit 1 = CUDA graph per step, bit 4 = generate() runs the prompt through the chunk path */
 jllm_b200_decoder* jllm_b200_decoder_create_layered(const jllm_b200_layered_desc* model, int flags);
 
+/* ── the mechanisms of layer-list models, one call each (extension) ─────────────────────────────────────
+ * kind: 2 = bf16, 3 = fp32 (weights, activations and caches).  Matrix rows and activation rows are padded to a multiple of 8
+ * elements (zeros), fp32 residual rows and norm vectors likewise. */
+/* Residual step of `rows` rows: x' = embed[tokens] | x + mult * LN(y; post), h = LN(x'; next).  y, or the weighted sum of
+ * expert rows sum_k weights[row][k] * y_exp[slots[row][k]], k < top.  x_out (optional) receives x'. */
+int jllm_b200_norm_step(void* h, float* x_out, const float* x, const float* y, const int* tokens, const void* embed, const void* y_exp, const int* slots,
+                        const float* weights, int top, const float* post_w, const float* post_b, const float* next_w, const float* next_b,
+                        float mult, float eps, int rows, int width, int kind, void* stream);
+/* Causal attention over caches [pos][n_kv_heads][head_dim] / [pos][n_kv_heads][v_dim] without rotation.  n_tokens > 0: queries
+ * at positions start .. start + n_tokens - 1; n_tokens = 0: one query over seq_len keys (n_splits KV slices, 0 = chosen).
+ * sink (optional): one logit per query head that joins the softmax denominator.  The scores of the query at position p carry
+ * the factor 1 + q_temp_coef * ln(floor((p + 1) / q_temp_every) + 1) (none for q_temp_every <= 0). */
+int jllm_b200_sink_attention(void* out, const void* q, const void* k, const void* v, int kind, int n_heads, int n_kv_heads, int head_dim, int v_dim,
+                             int n_tokens, int start, int seq_len, float scale, const float* sink, float q_temp_coef, double q_temp_every, int n_splits,
+                             void* stream);
+/* Routing of `rows` tokens from fp32 logits z [rows][n_experts]: s = sigmoid(z), choice = s + correction, groups of neighbouring
+ * experts ranked by their two largest choices, the top choices of the kept groups; ids, weights (= s), rank [rows][top] (place
+ * among the expert's tokens), counts [n_experts]. */
+int jllm_b200_moe_route(int* ids, float* weights, int* rank, int* counts, const float* z, const float* correction, int rows, int n_experts, int top,
+                        int n_groups, int keep_groups, void* stream);
+/* y[t][r] = W[r] . x[t]; with W_up, silu(W[r] . x[t]) * (W_up[r] . x[t]).  n_groups > 1: W holds n_groups matrices of M rows and
+ * group g takes token rows group_offsets[g] .. group_offsets[g + 1] - 1 (device array).  y rows: M fp32 or pad8(M) elements. */
+int jllm_b200_dense_matmul(void* y, const void* W, const void* W_up, const void* x, const int* group_offsets, int n_groups, int kind, int out_f32, int M,
+                           int N, int K, float softcap, void* stream);
+int jllm_b200_dense_matvec(void* y, const void* W, const void* x, int kind, int out_f32, int M, int K, float softcap, void* stream);
+/* One token through the chosen experts: routes it from z, act[k] = silu(gate . h) * (up . h), y = sum_k weights[k] * W_down . act[k] (fp32). */
+int jllm_b200_moe_matvec(void* y, void* act, int* ids, float* weights, const void* W_gate, const void* W_up, const void* W_down, const void* h,
+                         const float* z, const float* correction, int kind, int n_experts, int top, int n_groups, int keep_groups, int ff, int width,
+                         void* stream);
+
 /* ── tensor-parallel decoder session (extension; the reference is single-GPU) ───────────────────────────
  * One process per GPU.  Rank r of `world` (2, 4 or 8) owns rows [r*M/world, (r+1)*M/world) of every weight matrix
  * (a contiguous byte range of the GGUF image) and the KV heads that go with its query heads.  `model` carries the
