@@ -25,15 +25,21 @@ class JllmError(RuntimeError):
         self.code = code
 
 
+# the layer-list part of the library, which bin/trace_run builds in a checkout that has no complete library
+LAYERS_LIB_PATH = os.path.join(_HERE, "libjllm_b200_layers.so")
+
+
 def _load():
-    if not os.path.exists(LIB_PATH):
+    path = LIB_PATH if os.path.exists(LIB_PATH) or not os.path.exists(LAYERS_LIB_PATH) else LAYERS_LIB_PATH
+    if not os.path.exists(path):
         raise ImportError(
             f"{LIB_PATH} is missing: build it with `python genie-ai-runtime_b200/build.py` "
             "(nvcc, sm_100a). There is no fallback implementation.")
-    lib = C.CDLL(LIB_PATH)
+    lib = C.CDLL(path)
     lib.jllm_b200_last_error.restype = C.c_char_p
     lib.jllm_b200_launch_count.restype = C.c_longlong
-    lib.jllm_b200_get_splitk_partials.restype = C.c_void_p
+    if path == LIB_PATH:
+        lib.jllm_b200_get_splitk_partials.restype = C.c_void_p
     lib.jllm_b200_resolve_mapped_weight_device_ptr.restype = C.c_void_p
     for n in ("kv_pool_create", "kv_pool_key_ptr", "kv_pool_val_ptr", "kv_pool_scale_ptr", "scratch_create", "scratch_get"):
         getattr(lib, "jllm_b200_" + n).restype = C.c_void_p

@@ -5,6 +5,7 @@
 nvcc cross-compiles without a GPU; the resulting .so is what the tests, the smoke check
 and the benchmark load (there is no JIT and no fallback build at run time).
 """
+import fcntl
 import os
 import subprocess
 import sys
@@ -13,46 +14,72 @@ HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(HERE, "csrc")
 OUT = os.path.join(HERE, "libjllm_b200.so")
 NVCC = os.environ.get("NVCC", "/usr/local/cuda/bin/nvcc")
-SOURCES = ["core.cu", "api.cu", "gemv.cu", "elementwise.cu", "attention.cu", "attention_tma.cu", "attention_prefill.cu", "attention_noalloc.cu", "mmq.cu", "mmq_tc.cu", "mmq_stream.cu", "tp.cu", "decoder.cu", "decoder_kquant.cu", "decoder_layers.cu", "layernorm.cu", "dense_gemv.cu", "dense_simt.cu", "dense_tc.cu", "moe.cu", "attention_bf16.cu", "layers_api.cu", "batch_decoder.cu", "pools.cpp"]
+# What every model family needs, what the layer-list models add, and what the K-quant kernels and the reference's API add.
+COMMON = ["core.cu", "decoder.cu", "pools.cpp", "attention_general.cu"]
+LAYERS = ["decoder_layers.cu", "layernorm.cu", "dense_gemv.cu", "dense_simt.cu", "dense_tc.cu", "moe.cu", "attention_bf16.cu"]
+KQUANT = ["api.cu", "gemv.cu", "elementwise.cu", "attention.cu", "attention_tma.cu", "attention_prefill.cu", "attention_noalloc.cu", "mmq.cu", "mmq_tc.cu",
+          "mmq_stream.cu", "tp.cu", "decoder_kquant.cu", "batch_decoder.cu", "layers_api.cu"]
+SOURCES = COMMON + LAYERS + KQUANT
+# A command that serves one model in a fresh checkout builds only the part its architecture needs, as a library of its own.
+LAYERS_OUT = os.path.join(HERE, "libjllm_b200_layers.so")
+PARTS = {OUT: SOURCES, LAYERS_OUT: COMMON + LAYERS}
+ARCHITECTURE_LIBRARY = {"Ramilorn": LAYERS_OUT}
 FLAGS = ["-std=c++17", "-O3", "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo",
          "-Xcompiler", "-fPIC", "-Xcompiler", "-fvisibility=default", "--expt-relaxed-constexpr"]
 
 
-def sources():
-    return [os.path.join(CSRC, s) for s in SOURCES if os.path.exists(os.path.join(CSRC, s))]
+def sources(out=OUT):
+    return [os.path.join(CSRC, s) for s in PARTS[out]]
 
 
-def stale():
-    if not os.path.exists(OUT):
+def headers():
+    inc = os.path.join(HERE, "..", "include")
+    return [os.path.join(CSRC, h) for h in os.listdir(CSRC) if h.endswith((".cuh", ".h"))] + [os.path.join(inc, h) for h in os.listdir(inc)]
+
+
+def stale(out=OUT):
+    if not os.path.exists(out):
         return True
-    t = os.path.getmtime(OUT)
-    deps = [os.path.join(CSRC, f) for f in os.listdir(CSRC)] + [os.path.join(HERE, "..", "include", f) for f in os.listdir(os.path.join(HERE, "..", "include"))]
-    return any(os.path.getmtime(d) > t for d in deps)
+    t = os.path.getmtime(out)
+    return any(os.path.getmtime(d) > t for d in sources(out) + headers())
 
 
-def build_library(force=False, verbose=False):
-    if not force and not stale():
-        return OUT
+def build_library(force=False, verbose=False, out=OUT):
     objdir = os.path.join(HERE, "build")
     os.makedirs(objdir, exist_ok=True)
-    objs, procs = [], []
-    for src in sources():
-        obj = os.path.join(objdir, os.path.basename(src) + ".o")
-        objs.append(obj)
-        if not force and os.path.exists(obj) and os.path.getmtime(obj) > max(
-                os.path.getmtime(src), *[os.path.getmtime(os.path.join(CSRC, h)) for h in os.listdir(CSRC) if h.endswith((".cuh", ".h"))],
-                *[os.path.getmtime(os.path.join(HERE, "..", "include", h)) for h in os.listdir(os.path.join(HERE, "..", "include"))]):
-            continue
-        cmd = [NVCC] + FLAGS + (["-Xptxas", "-v"] if verbose else []) + ["-x", "cu", "-c", src, "-o", obj]
-        procs.append((src, subprocess.Popen(cmd, stdout=subprocess.PIPE, stderr=subprocess.STDOUT, text=True)))
-    for src, p in procs:
-        out, _ = p.communicate()
-        if p.returncode != 0:
-            raise RuntimeError(f"nvcc failed on {src}:\n{out}")
-        if verbose and out:
-            print(out)
-    subprocess.check_call([NVCC, "-shared", "-gencode", "arch=compute_100a,code=sm_100a", "-o", OUT] + objs + ["-lcudart"])
-    return OUT
+    with open(os.path.join(objdir, ".lock"), "w") as lock:      # one build of a checkout at a time
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        if not force and not stale(out):
+            return out
+        newest = max(os.path.getmtime(h) for h in headers())
+        objs, procs = [], []
+        for src in sources(out):
+            obj = os.path.join(objdir, os.path.basename(src) + ".o")
+            objs.append(obj)
+            if not force and os.path.exists(obj) and os.path.getmtime(obj) > max(os.path.getmtime(src), newest):
+                continue
+            cmd = [NVCC] + FLAGS + (["-Xptxas", "-v"] if verbose else []) + ["-x", "cu", "-c", src, "-o", obj]
+            procs.append((src, subprocess.Popen(cmd, stdout=subprocess.PIPE, stderr=subprocess.STDOUT, text=True)))
+        failed = []
+        for src, p in procs:
+            text, _ = p.communicate()
+            if p.returncode != 0:
+                failed.append(f"nvcc failed on {src}:\n{text}")
+            if verbose and text:
+                print(text)
+        if failed:
+            raise RuntimeError("\n".join(failed))
+        part = out + ".part"
+        subprocess.check_call([NVCC, "-shared", "-gencode", "arch=compute_100a,code=sm_100a", "-o", part] + objs + ["-lcudart"])
+        os.replace(part, out)
+        return out
+
+
+def ensure_library(architecture=None):
+    """Makes sure there is a library that serves `architecture` (None: everything): the complete one when it is there, else the
+    part the architecture needs.  Returns its path."""
+    out = OUT if os.path.exists(OUT) else ARCHITECTURE_LIBRARY.get(architecture, OUT)
+    return build_library(out=out)
 
 
 if __name__ == "__main__":

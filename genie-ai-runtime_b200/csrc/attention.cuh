@@ -37,6 +37,7 @@ bool   attention_prefill_fast_applies(const AttnCall& c);          // causal pre
 int    launch_attention_prefill_fast(const AttnCall& c, cudaStream_t st);
 bool   attention_bf16_applies(const AttnCall& c);                  // BF16 cache, head sizes multiples of 8 up to 256: decode and causal prefill
 int    launch_attention_bf16(const AttnCall& c, cudaStream_t st);
+int    launch_attention_float(const AttnCall& c, cudaStream_t st);    // BF16 and FP32 caches: the tensor-core kernels where they apply
 int    attn_bf16_splits(int seq_len, int n_heads, int n_kv);       // KV slices of a decode call at this length
 
 }  // namespace jb

@@ -432,4 +432,8 @@ int launch_attention_bf16(const AttnCall& c, cudaStream_t st) {
     return big <= 64 ? fa_launch<64>(a, prefill, st) : big <= 128 ? fa_launch<128>(a, prefill, st) : fa_launch<256>(a, prefill, st);
 }
 
+int launch_attention_float(const AttnCall& c, cudaStream_t st) {
+    return attention_bf16_applies(c) ? launch_attention_bf16(c, st) : launch_attention_general(c, st);
+}
+
 }  // namespace jb

@@ -1,0 +1,139 @@
+// attention_general.cu — decode / prefill attention over an FP16, INT8, BF16 or FP32 KV cache, sm_100a: the general kernel.
+//
+// Reference: src/kernels/attention.cu — single-query decode (:244-375), split-K partial +
+// reduce (:837-969), batched causal prefill (:382-514).  INT8 K/V carry one fp32 scale per
+// (position, kv head): k = k8*ks inside the QK dot, v = v8*vs inside PV.
+//
+// This file holds the general kernel: any head_dim <= 512, FP16, INT8, BF16 or FP32 cache, sliding
+// window, cache slot stride != head_dim, device-side position, ragged batches, causal prefill
+// (the slice itself is attention_general.cuh).  The tensor-core paths are attention_tma.cu and attention_prefill.cu (INT8,
+// 128-wide heads; chosen in attention.cu) and attention_bf16.cu.
+#include "attention.cuh"
+#include "attention_general.cuh"
+#include <cfloat>
+
+namespace jb {
+
+// Split policy (also what the decoder session keys its captured graphs on): one slice below 640 keys (a sliced call pays the
+// partials, a ticket and the merge), then slices of at least 128 keys (512 from 2048 keys on), at most 32 (the reference caps at
+// 8 slices for its 8-SM part, attention.cu:1000-1005).
+int attn_splits_for(int seq_len) {
+    if (seq_len < 640) return 1;
+    const int n = seq_len < 2048 ? seq_len / 128 : seq_len / 512;
+    return n > 32 ? 32 : n;
+}
+
+struct AttnArgs {
+    void* out; const void* q;
+    const void* k; const void* v; const float* ks; const float* vs;
+    // ragged batch (extension): per-sequence cache bases and lengths; null for one sequence
+    const void* const* k_list; const void* const* v_list; const float* const* ks_list; const float* const* vs_list;
+    const int* seq_lens;
+    int n_heads, n_kv, hd, chd, seq_len; const int* d_pos;
+    float scale; int kv_kind, window, n_splits;
+    int causal_start;       // prefill: query t sees start+t+1 keys (blockIdx.z = t); -1 = decode
+    float* part;            // [z][head][split] m | l | acc[vhd]
+    int vhd, ldq, ldo;      // value head size, row strides of q and out
+    const float* sink; float qt_coef; double qt_every;
+};
+
+// QT: type of q and of the output
+template <typename QT>
+__global__ void __launch_bounds__(AG_THREADS) attn_general_kernel(const AttnArgs a) {
+    pdl_wait();
+    extern __shared__ float sm[];
+    const int head = blockIdx.x, split = blockIdx.y, z = blockIdx.z;
+    const int kvh = head / (a.n_heads / a.n_kv);
+    AgCache c = { a.k, a.v, a.ks, a.vs, a.n_kv, a.chd, a.kv_kind, a.window, a.vhd };
+    int seq = a.d_pos ? (*a.d_pos + 1) : a.seq_len;
+    if (a.k_list) { c.k = a.k_list[z]; c.v = a.v_list[z]; c.ks = a.ks_list ? a.ks_list[z] : nullptr; c.vs = a.vs_list ? a.vs_list[z] : nullptr; seq = a.seq_lens[z]; }
+    if (a.causal_start >= 0) seq = a.causal_start + z + 1;
+    const int per = (seq + a.n_splits - 1) / a.n_splits, vhd = a.vhd > 0 ? a.vhd : a.hd;
+    const int kv0 = split * per, kv1 = min(kv0 + per, seq);
+    const QT* q = reinterpret_cast<const QT*>(a.q) + (size_t)z * a.ldq + (size_t)head * a.hd;
+    QT* out = reinterpret_cast<QT*>(a.out) + (size_t)z * a.ldo + (size_t)head * vhd;
+    const float scale = a.scale * q_temp_factor(seq - 1, a.qt_coef, a.qt_every);
+    float M, L;
+    if (a.n_splits == 1) {
+        // emit() runs after M and L are final, so the normalisation can be applied on the way out
+        ag_slice(q, c, kvh, a.hd, seq, kv0, kv1, scale, sm, M, L,
+                 [&](int d, float o) { out[d] = from_f32<QT>(o * sink_norm(M, L, a.sink ? a.sink + head : nullptr)); });
+    } else {
+        float* pb = a.part + (((size_t)z * a.n_heads + head) * a.n_splits + split) * (vhd + 2);
+        ag_slice(q, c, kvh, a.hd, seq, kv0, kv1, scale, sm, M, L, [&](int d, float o) { pb[2 + d] = o; });
+        if (threadIdx.x == 0) { pb[0] = L > 0.f ? M : -FLT_MAX; pb[1] = L; }
+    }
+}
+
+template <typename QT>
+__global__ void attn_reduce_kernel(QT* out, const float* part, int n_heads, int hd, int n_splits, int ldo, const float* sink) {
+    pdl_wait();
+    const int head = blockIdx.x, z = blockIdx.y;
+    ag_merge_slices(out + (size_t)z * ldo + (size_t)head * hd, part + ((size_t)z * n_heads + head) * n_splits * (hd + 2), hd, n_splits, sink ? sink + head : nullptr);
+}
+
+float* splitk_buffer(size_t floats, bool may_alloc) {
+    DeviceCtx* c = ctx();
+    if (!c) return nullptr;
+    if (floats > c->splitk_floats) {
+        if (!may_alloc) return nullptr;
+        if (c->splitk) cudaFree(c->splitk);
+        c->splitk = nullptr; c->splitk_floats = 0;
+        if (cudaMalloc(&c->splitk, floats * sizeof(float)) != cudaSuccess) { cudaGetLastError(); return nullptr; }
+        c->splitk_floats = floats;
+    }
+    return c->splitk;
+}
+
+static bool stream_capturing(cudaStream_t st) {
+    cudaStreamCaptureStatus cs = cudaStreamCaptureStatusNone;
+    if (cudaStreamIsCapturing(st, &cs) != cudaSuccess) { cudaGetLastError(); return false; }
+    return cs != cudaStreamCaptureStatusNone;
+}
+
+int launch_attention_general(const AttnCall& c, cudaStream_t st) {
+    if (c.n_heads <= 0 || c.n_kv <= 0 || c.n_heads % c.n_kv) return set_error(JB_ERR_ARG, "attention: n_heads=%d n_kv_heads=%d", c.n_heads, c.n_kv);
+    if (c.hd <= 0 || c.hd > 512 || c.chd < c.hd) return set_error(JB_ERR_ARG, "attention: head_dim=%d cache_head_dim=%d", c.hd, c.chd);
+    if (!c.out || !c.q) return set_error(JB_ERR_PTR, "attention: null q/out");
+    if (!c.k_list && (!c.k || !c.v)) return set_error(JB_ERR_PTR, "attention: null cache pointer");
+    const int batch = c.batch > 0 ? c.batch : 1, vhd = c.vhd > 0 ? c.vhd : c.hd;
+    if (vhd > 512) return set_error(JB_ERR_ARG, "attention: value head_dim=%d", vhd);
+    int n_splits = c.n_splits > 0 ? c.n_splits : (c.d_pos || c.causal_start >= 0 ? 1 : attn_splits_for(c.k_list ? c.max_seq : c.seq_len));
+    if (!c.d_pos && !c.k_list && c.causal_start < 0 && c.seq_len <= 0) {     // nothing to attend to: zeros, like an empty softmax
+        JB_CUDA(cudaMemsetAsync(c.out, 0, (size_t)c.n_heads * vhd * (c.kind() == EK_F32 ? 4 : 2), st));
+        return JB_OK;
+    }
+    AttnArgs a = {};
+    a.out = c.out; a.q = c.q; a.k = c.k; a.v = c.v; a.ks = c.ks; a.vs = c.vs;
+    a.k_list = c.k_list; a.v_list = c.v_list; a.ks_list = c.ks_list; a.vs_list = c.vs_list; a.seq_lens = c.seq_lens;
+    a.n_heads = c.n_heads; a.n_kv = c.n_kv; a.hd = c.hd; a.chd = c.chd; a.seq_len = c.seq_len; a.d_pos = c.d_pos;
+    a.vhd = c.vhd; a.ldq = c.ldq > 0 ? c.ldq : c.n_heads * c.hd; a.ldo = c.ldo > 0 ? c.ldo : c.n_heads * vhd;
+    a.sink = c.sink; a.qt_coef = c.qt_coef; a.qt_every = c.qt_every;
+    a.scale = c.scale; a.kv_kind = c.kind(); a.window = c.window; a.causal_start = c.causal_start;
+    if (n_splits > 1) {
+        const size_t need = (size_t)batch * c.n_heads * n_splits * (vhd + 2);
+        a.part = splitk_buffer(need, !stream_capturing(st));
+        if (!a.part) n_splits = 1;       // no scratch (or capture in progress): one slice per head, still on the GPU
+    }
+    a.n_splits = n_splits;
+    const dim3 grid(c.n_heads, n_splits, batch);
+    const size_t smem = ag_smem_bytes(vhd);
+    switch (c.kind()) {
+        case EK_BF16: JB_CUDA(launch_k(attn_general_kernel<__nv_bfloat16>, grid, dim3(AG_THREADS), smem, st, pdl_enabled(), a)); break;
+        case EK_F32:  JB_CUDA(launch_k(attn_general_kernel<float>, grid, dim3(AG_THREADS), smem, st, pdl_enabled(), a)); break;
+        default:      JB_CUDA(launch_k(attn_general_kernel<__half>, grid, dim3(AG_THREADS), smem, st, pdl_enabled(), a));
+    }
+    count_launch();
+    if (n_splits > 1) {
+        const dim3 rg(c.n_heads, batch);
+        switch (c.kind()) {
+            case EK_BF16: JB_CUDA(launch_k(attn_reduce_kernel<__nv_bfloat16>, rg, dim3(128), 0, st, pdl_enabled(), (__nv_bfloat16*)c.out, (const float*)a.part, c.n_heads, vhd, n_splits, a.ldo, c.sink)); break;
+            case EK_F32:  JB_CUDA(launch_k(attn_reduce_kernel<float>, rg, dim3(128), 0, st, pdl_enabled(), (float*)c.out, (const float*)a.part, c.n_heads, vhd, n_splits, a.ldo, c.sink)); break;
+            default:      JB_CUDA(launch_k(attn_reduce_kernel<__half>, rg, dim3(128), 0, st, pdl_enabled(), (__half*)c.out, (const float*)a.part, c.n_heads, vhd, n_splits, a.ldo, c.sink));
+        }
+        count_launch();
+    }
+    return JB_OK;
+}
+
+}  // namespace jb

@@ -134,7 +134,7 @@ int LayerDecoder::enqueue_step(int n_splits, cudaStream_t st) {
         DCHK(launch_dense_gemv(g, st));
         AttnCall c = attention_call(l, a);
         c.d_pos = d_pos; c.n_splits = n_splits;
-        DCHK(launch_attention(c, st));
+        DCHK(launch_attention_float(c, st));
         DenseGemv o;
         o.kind = kind; o.W = w.w_o; o.M = m.width; o.K = w.n_heads * w.v_dim; o.x = a.att; o.seg[0] = OutSeg{a.y, pad8(m.width), m.width, 1, 0};
         DCHK(launch_dense_gemv(o, st));
@@ -193,7 +193,7 @@ int LayerDecoder::enqueue_chunk(const int* dev_tokens, int N, int start, cudaStr
         DCHK(launch_dense_gemm(g, st));
         AttnCall c = attention_call(l, a);
         c.causal_start = start; c.batch = N; c.n_splits = 1;
-        DCHK(launch_attention(c, st));
+        DCHK(launch_attention_float(c, st));
         DenseGemm o;
         o.kind = kind; o.W = w.w_o; o.M = m.width; o.K = w.n_heads * w.v_dim; o.N = N; o.x = a.att; o.seg[0] = OutSeg{a.y, pad8(m.width), m.width, 1, 0};
         DCHK(launch_dense_gemm(o, st));

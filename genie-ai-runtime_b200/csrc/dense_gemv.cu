@@ -1,7 +1,8 @@
 // dense_gemv.cu — one token against dense weights: the decode products of layer-list models, HBM-bound.
 //
-// Two CTAs of eight warps per SM; the output rows (or gate / up row pairs) are dealt to the warps in contiguous runs, a
-// warp walks R rows at a time and keeps eight 16-byte weight loads per lane in flight, one batch ahead of the arithmetic.
+// Two CTAs of eight warps per SM; the output rows (or gate / up row pairs) are dealt to the CTAs in contiguous runs and
+// within a CTA to groups of 1, 2, 4 or 8 warps that share a row (as many as make the warps' work most even).  A warp walks R
+// rows at a time and keeps eight 16-byte weight loads per lane in flight, one batch ahead of the arithmetic.
 // Where the rows do not depend on the previous kernel (all modes but the expert ones) the first batch is requested before
 // griddepcontrol.wait, so the weights stream in while the input vector is still being produced and normed.  The input
 // vector is held in shared memory in the activation type (what the prompt path multiplies), sums are fp32.
@@ -29,44 +30,54 @@ struct DgArgs {
     DenseGemv g;
     int nchunk;          // 16-byte chunks of the input vector (of one expert's input for GEMV_MOE_DOWN)
     uint32_t magic;      // ceil(2^32 / nchunk): chunk / nchunk by one multiply
+    int split;           // warps that share a row (1, 2, 4 or 8), each with its range of chunks
+    int off_part;        // shared memory: start of the partial sums
 };
 
 template <typename T, int MODE, int R>
 __global__ void __launch_bounds__(DG_THREADS, 2) dense_gemv_kernel(const DgArgs p) {
     constexpr int U = DG_LOADS / R;              // chunks per row in a batch
+    constexpr int STEP = MODE == GEMV_MOE_UP ? 1 : R;                 // items per group of rows (an up item is two rows)
     extern __shared__ __align__(16) unsigned char dg_sm[];
-    __shared__ float red[DG_WARPS];
+    __shared__ float red[NORM_RED * DG_WARPS];
     __shared__ int s_ids[MOE_MAX_TOP];
     __shared__ float s_wts[MOE_MAX_TOP];
     const DenseGemv& g = p.g;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const int total_warps = gridDim.x * DG_WARPS, wid = blockIdx.x * DG_WARPS + warp;
     const int items = MODE == GEMV_MOE_UP ? g.route.top * g.M : g.M;
-    const int r0 = (int)((long long)items * wid / total_warps), r1 = (int)((long long)items * (wid + 1) / total_warps);
-    constexpr int STEP = MODE == GEMV_MOE_UP ? 1 : R;                 // items per group (an up item is two rows)
+    // this CTA's items [i0, i1); warp (grp, part) takes items i0 + grp, + groups, ... and chunks [c0, c1) of each
+    const int i0 = (int)((long long)items * blockIdx.x / gridDim.x), i1 = (int)((long long)items * (blockIdx.x + 1) / gridDim.x);
+    const int groups = DG_WARPS / p.split, grp = warp / p.split, part = warp - grp * p.split;
+    const int mine = i1 - i0 > grp ? (i1 - i0 - grp + groups - 1) / groups : 0;
     const int nchunk = MODE == GEMV_MOE_DOWN ? p.nchunk * g.route.top : p.nchunk;
-    const int nb = (nchunk + 32 * U - 1) / (32 * U);
-    const int n_batches = r1 > r0 ? ((r1 - r0 + STEP - 1) / STEP) * nb : 0;
+    const int c0 = (int)((long long)nchunk * part / p.split), c1 = (int)((long long)nchunk * (part + 1) / p.split);
+    const int nb = (c1 - c0 + 32 * U - 1) / (32 * U);
+    const int n_batches = ((mine + STEP - 1) / STEP) * nb;
     uint4* hs = reinterpret_cast<uint4*>(dg_sm);
+    float* partial = reinterpret_cast<float*>(dg_sm + p.off_part);
 
-    auto load = [&](int item, int b, uint4 (&w)[DG_LOADS]) {
+    auto item_at = [&](int j) { return i0 + grp + min(j, mine - 1) * groups; };
+    auto load = [&](int j, int b, uint4 (&w)[DG_LOADS]) {             // batch b of the rows of the warp's items j .. j + STEP - 1
         #pragma unroll
         for (int r = 0; r < R; ++r) {
             const uint4* row = nullptr;
+            int item = 0;
             if (MODE == GEMV_MOE_UP) {
+                item = item_at(j);
                 const int k = item / g.M, f = item - k * g.M;
                 row = reinterpret_cast<const uint4*>(r == 0 ? g.W : g.W_up) + ((size_t)s_ids[k] * g.M + f) * p.nchunk;
-            } else if (MODE != GEMV_MOE_DOWN) {
-                row = reinterpret_cast<const uint4*>(g.W) + (size_t)min(item + r, r1 - 1) * p.nchunk;
+            } else {
+                item = item_at(j + r);
+                row = reinterpret_cast<const uint4*>(g.W) + (size_t)item * p.nchunk;
             }
             #pragma unroll
             for (int u = 0; u < U; ++u) {
-                const int c = (b * U + u) * 32 + lane;
+                const int c = c0 + (b * U + u) * 32 + lane;
                 w[r * U + u] = make_uint4(0, 0, 0, 0);
-                if (c < nchunk) {
+                if (c < c1) {
                     if (MODE == GEMV_MOE_DOWN) {
-                        const int k = p.nchunk == 1 ? c : (int)__umulhi((uint32_t)c, p.magic), cc = c - k * p.nchunk;
-                        w[r * U + u] = __ldg(reinterpret_cast<const uint4*>(g.W) + ((size_t)s_ids[k] * g.M + min(item + r, r1 - 1)) * p.nchunk + cc);
+                        const int k = p.nchunk == 1 ? c : (int)__umulhi((uint32_t)c, p.magic);
+                        w[r * U + u] = __ldg(row + (size_t)s_ids[k] * g.M * p.nchunk + (c - k * p.nchunk));
                     } else {
                         w[r * U + u] = __ldg(row + c);
                     }
@@ -74,9 +85,18 @@ __global__ void __launch_bounds__(DG_THREADS, 2) dense_gemv_kernel(const DgArgs 
             }
         }
     };
+    auto finish = [&](int item, float v, float v2) {
+        if (MODE == GEMV_MOE_UP) {
+            const int k = item / g.M, f = item - k * g.M;
+            reinterpret_cast<T*>(g.seg[0].y)[(long long)k * g.seg[0].ld + f] = from_f32<T>(silu_f(v) * v2);
+        } else {
+            store_seg<T>(g.seg, g.nseg, g.softcap, g.d_pos, 0, item, v);
+        }
+    };
 
     uint4 cur[DG_LOADS], nxt[DG_LOADS];
-    if (MODE == GEMV_NORM || MODE == GEMV_PLAIN) { if (n_batches > 0) load(r0, 0, cur); }
+    if (MODE == GEMV_NORM || MODE == GEMV_PLAIN) { if (n_batches > 0) load(0, 0, cur); }
+    if (MODE == GEMV_NORM) norm_prefetch<DG_THREADS>(g.norm);
     pdl_wait();
     pdl_launch();
     // ── the input vector ──
@@ -101,21 +121,21 @@ __global__ void __launch_bounds__(DG_THREADS, 2) dense_gemv_kernel(const DgArgs 
             for (int k = threadIdx.x; k < g.route.top; k += DG_THREADS) { s_ids[k] = g.ids[k]; s_wts[k] = g.wts[k]; }
         }
         __syncthreads();
-        if (MODE != GEMV_PLAIN && n_batches > 0) load(r0, 0, cur);
+        if (MODE != GEMV_PLAIN && n_batches > 0) load(0, 0, cur);
     }
     // ── the products ──
     float acc[R];
     #pragma unroll
     for (int r = 0; r < R; ++r) acc[r] = 0.f;
-    int item = r0, b = 0;
+    int j = 0, b = 0;
     for (int it = 0; it < n_batches; ++it) {
-        int item_n = item, b_n = b + 1;
-        if (b_n == nb) { b_n = 0; item_n += STEP; }
-        if (it + 1 < n_batches) load(item_n, b_n, nxt);
+        int j_n = j, b_n = b + 1;
+        if (b_n == nb) { b_n = 0; j_n += STEP; }
+        if (it + 1 < n_batches) load(j_n, b_n, nxt);
         #pragma unroll
         for (int u = 0; u < U; ++u) {
-            const int c = (b * U + u) * 32 + lane;
-            if (c < nchunk) {
+            const int c = c0 + (b * U + u) * 32 + lane;
+            if (c < c1) {
                 const uint4 h = hs[c];
                 if (MODE == GEMV_MOE_DOWN) {
                     const float w = s_wts[p.nchunk == 1 ? c : (int)__umulhi((uint32_t)c, p.magic)];
@@ -130,22 +150,34 @@ __global__ void __launch_bounds__(DG_THREADS, 2) dense_gemv_kernel(const DgArgs 
         if (b_n == 0) {
             #pragma unroll
             for (int r = 0; r < R; ++r) acc[r] = warp_sum(acc[r]);
-            if (MODE == GEMV_MOE_UP) {
-                if (lane == 0) {
-                    const int k = item / g.M, f = item - k * g.M;
-                    reinterpret_cast<T*>(g.seg[0].y)[(long long)k * g.seg[0].ld + f] = from_f32<T>(silu_f(acc[0]) * acc[R > 1 ? 1 : 0]);
-                }
-            } else {
+            if (p.split > 1) {
                 #pragma unroll
                 for (int r = 0; r < R; ++r)
-                    if (lane == r && item + r < r1) store_seg<T>(g.seg, g.nseg, g.softcap, g.d_pos, 0, item + r, acc[r]);
+                    if (lane == r && (MODE == GEMV_MOE_UP || j + r < mine))
+                        partial[((item_at(MODE == GEMV_MOE_UP ? j : j + r) - i0) * p.split + part) * (MODE == GEMV_MOE_UP ? 2 : 1) + (MODE == GEMV_MOE_UP ? r : 0)] = acc[r];
+            } else if (MODE == GEMV_MOE_UP) {
+                if (lane == 0) finish(item_at(j), acc[0], acc[R > 1 ? 1 : 0]);
+            } else {
+                #pragma unroll
+                for (int r = 0; r < R; ++r) if (lane == r && j + r < mine) finish(item_at(j + r), acc[r], 0.f);
             }
             #pragma unroll
             for (int r = 0; r < R; ++r) acc[r] = 0.f;
         }
         #pragma unroll
         for (int i = 0; i < DG_LOADS; ++i) cur[i] = nxt[i];
-        item = item_n; b = b_n;
+        j = j_n; b = b_n;
+    }
+    if (p.split > 1) {                           // partial sums of a row in the order of its chunks
+        __syncthreads();
+        for (int i = threadIdx.x; i < i1 - i0; i += DG_THREADS) {
+            float v = 0.f, v2 = 0.f;
+            for (int q = 0; q < p.split; ++q) {
+                if (MODE == GEMV_MOE_UP) { v += partial[(i * p.split + q) * 2]; v2 += partial[(i * p.split + q) * 2 + 1]; }
+                else v += partial[i * p.split + q];
+            }
+            finish(i0 + i, v, v2);
+        }
     }
 }
 
@@ -188,15 +220,27 @@ int launch_dense_gemv(const DenseGemv& a, cudaStream_t st) {
     p.nchunk = pad8(a.K) * es / 16;
     p.magic = p.nchunk > 1 ? (uint32_t)((0x100000000ull + p.nchunk - 1) / p.nchunk) : 0;
     const int chunks = a.mode == GEMV_MOE_DOWN ? p.nchunk * a.route.top : p.nchunk;
+    const int items = a.mode == GEMV_MOE_UP ? a.route.top * a.M : a.M;
+    const int grid = items < 2 * c->sm_count ? items : 2 * c->sm_count, per_cta = (items + grid - 1) / grid;
+    // warps per row and rows at a time: the fewest loads of the busiest warp (slots of a batch that a row does not fill count a
+    // little: they cost no traffic, but leave less in flight; so do the reduction at the end of a row and a split)
+    int R = 1;
+    double best = 1e30;
+    for (int S = 1; S <= DG_WARPS; S *= 2) {
+        const int rows = (per_cta + DG_WARPS / S - 1) / (DG_WARPS / S), lanes = ((chunks + S - 1) / S + 31) / 32;
+        for (int r = a.mode == GEMV_MOE_UP ? 2 : 1; r <= (a.mode == GEMV_MOE_UP ? 2 : 4); r *= 2) {
+            const int u = DG_LOADS / r, step = a.mode == GEMV_MOE_UP ? 1 : r, trips = (rows + step - 1) / step, nb = (lanes + u - 1) / u;
+            const double used = (double)trips * r * lanes, slots = (double)trips * r * nb * u;
+            const double cost = used + 0.5 * (slots - used) + 1.0 * trips + (S > 1 ? 2.0 : 0.0);
+            if (cost < best - 1e-9) { best = cost; R = r; p.split = S; }
+        }
+    }
     size_t smem = (size_t)chunks * 16;
     if (a.mode == GEMV_NORM) smem += (size_t)pad8(a.K) * 4;
-    if (a.mode == GEMV_MOE_UP) smem += (size_t)(2 * a.route.n_experts + a.route.n_groups) * 4;
+    if (a.mode == GEMV_MOE_UP) smem += ((size_t)(2 * a.route.n_experts + a.route.n_groups) * 4 + 15) & ~(size_t)15;
+    p.off_part = (int)smem;
+    if (p.split > 1) smem += (size_t)per_cta * p.split * (a.mode == GEMV_MOE_UP ? 8 : 4);
     if (smem > (size_t)c->max_smem_optin - 2048) return set_error(JB_ERR_LIMIT, "dense gemv: input of %d elements", a.K);
-    const int items = a.mode == GEMV_MOE_UP ? a.route.top * a.M : a.M;
-    const int full = 2 * c->sm_count, per_warp = items / (full * DG_WARPS);
-    const int R = per_warp >= 4 ? 4 : per_warp >= 2 ? 2 : 1;
-    const int want = (items + DG_WARPS - 1) / DG_WARPS;
-    const int grid = want < full ? want : full;
     return a.kind == EK_F32 ? dg_mode<float>(p, R, grid, smem, st) : dg_mode<__nv_bfloat16>(p, R, grid, smem, st);
 }
 

@@ -9,7 +9,7 @@ template <typename T>
 __global__ void __launch_bounds__(NR_THREADS) norm_rows_kernel(const NormStep a) {
     pdl_wait();
     extern __shared__ __align__(16) float nr_buf[];
-    __shared__ float red[NR_THREADS / 32];
+    __shared__ float red[NORM_RED * NR_THREADS / 32];
     const int row = blockIdx.x;
     norm_step_row<T, NR_THREADS>(a, row, nr_buf, red, a.x_out != nullptr, reinterpret_cast<T*>(a.h) + (size_t)row * pad8(a.W));
 }

@@ -11,6 +11,7 @@
 
 namespace jb {
 
+constexpr int NORM_RED = 4;              // reduction words per warp of a residual step
 constexpr int EK_F16 = 0, EK_INT8 = 1, EK_BF16 = 2, EK_F32 = 3;      // element kinds of caches and activations
 inline int elem_bytes(int kind) { return kind == EK_F32 ? 4 : kind == EK_INT8 ? 1 : 2; }
 __host__ __device__ inline int pad8(int n) { return (n + 7) & ~7; }
@@ -48,7 +49,7 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
     *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
 }
 
-// sum over the CTA, the same value on every thread; red: THREADS / 32 floats
+// sum over the CTA, the same value on every thread; red: THREADS / 32 floats that the CTA's next sum must not share
 template <int THREADS>
 __device__ __forceinline__ float block_sum(float v, float* red) {
     v = warp_sum(v);
@@ -57,10 +58,9 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
     float s = 0.f;
     #pragma unroll
     for (int i = 0; i < THREADS / 32; ++i) s += red[i];
-    __syncthreads();
     return s;
 }
-// mean and 1/sqrt(var + eps) of buf[0..W)
+// mean and 1/sqrt(var + eps) of buf[0..W); red: 2 * THREADS / 32 floats
 template <int THREADS>
 __device__ __forceinline__ void ln_stats(const float* buf, int W, float eps, float* red, float& mean, float& rstd) {
     const int n4 = pad8(W) / 4;
@@ -74,10 +74,26 @@ __device__ __forceinline__ void ln_stats(const float* buf, int W, float eps, flo
         #pragma unroll
         for (int e = 0; e < 4; ++e) if (4 * i + e < W) q = fmaf(d[e], d[e], q);
     }
-    rstd = 1.0f / sqrtf(block_sum<THREADS>(q, red) / (float)W + eps);
+    rstd = 1.0f / sqrtf(block_sum<THREADS>(q, red + THREADS / 32) / (float)W + eps);
+}
+// Requests the rows a residual step will read that no kernel still running writes: the norm vectors (constants), and the
+// residual row, whose producer finished before the kernel in front of this one started.
+template <int THREADS>
+__device__ __forceinline__ void norm_prefetch(const NormStep& a) {
+    const int lines = (pad8(a.W) * 4 + 127) / 128;
+    for (int i = threadIdx.x; i < lines; i += THREADS) {
+        const size_t o = (size_t)i * 32;
+        asm volatile("prefetch.global.L1 [%0];" ::"l"(a.next_w + o));
+        asm volatile("prefetch.global.L1 [%0];" ::"l"(a.next_b + o));
+        if (!a.tokens) {
+            asm volatile("prefetch.global.L1 [%0];" ::"l"(a.post_w + o));
+            asm volatile("prefetch.global.L1 [%0];" ::"l"(a.post_b + o));
+            asm volatile("prefetch.global.L1 [%0];" ::"l"(a.x + o));
+        }
+    }
 }
 // One row by the whole CTA.  buf: pad8(W) floats of shared memory (each thread touches only its own elements of it);
-// red: THREADS / 32 floats; h_out: where the normed row goes (shared or global).
+// red: NORM_RED floats per warp of the CTA; h_out: where the normed row goes (shared or global).
 template <typename T, int THREADS>
 __device__ __forceinline__ void norm_step_row(const NormStep& a, int row, float* buf, float* red, bool write_x, T* h_out) {
     const int ld = pad8(a.W), n4 = ld / 4, src = a.row_index ? a.row_index[row] : row;
@@ -104,7 +120,7 @@ __device__ __forceinline__ void norm_step_row(const NormStep& a, int row, float*
             for (int i = threadIdx.x; i < n4; i += THREADS) store4(buf + 4 * i, load4(a.y + off + 4 * i));
         }
         float mean, rstd;
-        ln_stats<THREADS>(buf, a.W, a.eps, red, mean, rstd);
+        ln_stats<THREADS>(buf, a.W, a.eps, red + 2 * THREADS / 32, mean, rstd);
         for (int i = threadIdx.x; i < n4; i += THREADS) {
             const float4 v = load4(buf + 4 * i), x = load4(a.x + off + 4 * i), w = load4(a.post_w + 4 * i), b = load4(a.post_b + 4 * i);
             float4 r;
