@@ -1,6 +1,6 @@
 // attention_general.cuh — the general attention slice: one query head against keys [kv0, kv1) of an FP16, INT8, BF16 or
 // FP32 cache of any head size up to 512 (values may have their own), optional sliding window, cache slot stride >= head
-// size, optional softmax sink (one more term in the denominator, no key and no value).
+// size, optional softmax sink (a logit that joins the denominator only).
 //
 // Same mathematics as the reference's decode / split-K / prefill kernels (src/kernels/attention.cu:244-375, :382-514,
 // :837-941: s_j = scale * q . k_j with k = k8 * ks for INT8, online softmax, o = Σ p_j v_j with v = v8 * vs), arranged

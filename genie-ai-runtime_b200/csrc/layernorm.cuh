@@ -2,7 +2,7 @@
 //     x' = embed[token]                      (start of the stack)
 //     x' = x + mult * LN(y; post)            (exit of a sublayer, normed before it is added)
 //     h  = LN(x'; next)                      (entry of the next sublayer)
-// with LN(v; w, b) = (v - mean) / sqrt(var + eps) * w + b, var the mean of the squared deviations.  All of it in fp32; h is
+// with LN(v; w, b) = (v - mu) / sqrt(s2 + eps) * w + b, mu = mean(v), s2 = mean((v - mu)^2).  All of it in fp32; h is
 // rounded to the activation type.  The same device function serves the row kernel of the prompt path (layernorm.cu) and
 // the prologue of the decode products (dense_gemv.cu), so both give the same bits.
 #pragma once

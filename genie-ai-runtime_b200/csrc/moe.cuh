@@ -1,6 +1,6 @@
 // moe.cuh — mixture-of-experts routing: sigmoid scores, a per-expert correction that enters the choice only, optional
-// groups of neighbouring experts of which the best few stay eligible (a group's score is the sum of its two largest
-// choice scores), the `top` largest choice scores among the eligible, weights = the uncorrected scores.
+// groups of consecutive experts of which a few stay eligible (ranked by best + second-best choice score of the group),
+// the `top` largest choice scores among the eligible, weights = the scores without correction.
 #pragma once
 #include "layernorm.cuh"
 

@@ -40,7 +40,7 @@ def random_model(jb, s, dev, seed=7):
     w = L.LayeredWeights.__new__(L.LayeredWeights)
     layers = [L.LayerSpec(L.AttentionSpec(s["heads"], s["kv_heads"], s["dim"], s["vdim"], s["dim"] ** -0.5, -1, 0.1, 4096.0),
                           L.MoeSpec(s["experts"], s["top"], s["ff"], s["groups"], s["keep"])) for _ in range(s["n_layers"])]
-    w.cfg = L.LayeredConfig(vocab=s["vocab"], width=W, layers=layers, eps=1e-5, residual_mult=0.5, logit_softcap=30.0)
+    w.cfg = L.LayeredConfig(vocab=s["vocab"], width=W, layers=layers, eps=1e-6, residual_mult=0.6, logit_softcap=40.0)
     w.dtype = "bfloat16"
     norm = lambda f: {f + "_w": vec(W, 1.0), f + "_b": vec(W, 0.0)}
     w.top = {"embed": torch.randn((s["vocab"], W), device=dev, generator=g, dtype=dt), **norm("final")}

@@ -1,10 +1,10 @@
 """Replays a token trace through a model and writes logits: `bin/trace_run --model DIR --dtype bfloat16|float32 --out DIR
 --max-tokens N`.
 
-Standard input carries one step per line, {"step": n, "entries": [{"id": ..., "tokens": [...], "want": [...]}], "end": [...]}:
-the next tokens of requests and the places among them whose logits are wanted, then the requests that are finished.  A
-step with wanted places writes <out>/<n>.f32 (float32 rows in the order of entries and places); every step prints `done n`.
-Exit code 3: the model does not run in the requested number format.
+Standard input is JSON lines, {"step": n, "entries": [{"id": ..., "tokens": [...], "want": [...]}], "end": [...]}: an entry
+appends tokens to a request and lists the indices into them that need logits; `end` names requests to release.  Logits go to
+<out>/<n>.f32 (float32 rows, entry by entry, index by index), no file for a step that needs none; `done n` is printed after
+each step.  Exit code 3: the model does not run in the requested number format.
 """
 from __future__ import annotations
 
@@ -38,7 +38,7 @@ def main(argv=None):
     ap.add_argument("--model", required=True, help="folder with config.json and model.safetensors")
     ap.add_argument("--dtype", required=True, help="number format, e.g. bfloat16 or float32")
     ap.add_argument("--out", required=True, help="folder for the <step>.f32 files")
-    ap.add_argument("--max-tokens", type=int, required=True, help="most tokens that live requests hold at any time")
+    ap.add_argument("--max-tokens", type=int, required=True, help="cache size: positions a request may fill")
     a = ap.parse_args(argv)
     try:
         check_config(read_config(a.model), a.dtype)

@@ -329,8 +329,8 @@ int jllm_b200_norm_step(void* h, float* x_out, const float* x, const float* y, c
 int jllm_b200_sink_attention(void* out, const void* q, const void* k, const void* v, int kind, int n_heads, int n_kv_heads, int head_dim, int v_dim,
                              int n_tokens, int start, int seq_len, float scale, const float* sink, float q_temp_coef, double q_temp_every, int n_splits,
                              void* stream);
-/* Routing of `rows` tokens from fp32 logits z [rows][n_experts]: s = sigmoid(z), choice = s + correction, groups of neighbouring
- * experts ranked by their two largest choices, the top choices of the kept groups; ids, weights (= s), rank [rows][top] (place
+/* Routing of `rows` tokens from fp32 logits z [rows][n_experts]: s = sigmoid(z), choice = s + correction, groups of
+ * consecutive experts ranked by best + second-best choice, the top choices of the kept groups; ids, weights (= s), rank [rows][top] (place
  * among the expert's tokens), counts [n_experts]. */
 int jllm_b200_moe_route(int* ids, float* weights, int* rank, int* counts, const float* z, const float* correction, int rows, int n_experts, int top,
                         int n_groups, int keep_groups, void* stream);

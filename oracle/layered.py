@@ -1,6 +1,6 @@
 """Plain restatement of the layer-list decoder models (Ramilorn), one function per mechanism, in float64 numpy.
 
-The checker of the layer-list path: slow, no cache, no batching, nothing shared with the library.  A model is its
+The oracle of the layer-list path: slow, no cache, no batching, nothing shared with the library.  A model is its
 configuration dict (the parsed config.json) and a dict of tensors by name.  All functions take and return float64
 arrays; a sequence is a [tokens, width] array.
 """

@@ -21,7 +21,7 @@ def moe(experts, top, ff, groups=None):
     return dict(kind="moe", expert=dict(ff=ff), router=r)
 
 
-def config(vocab, width, layers, eps=1e-5, mult=0.5, softcap=30.0):
+def config(vocab, width, layers, eps=1e-4, mult=0.8, softcap=25.0):
     c = dict(architecture="Ramilorn", vocab=vocab, width=width, norm=dict(eps=eps), residual_mult=mult,
              layers=[dict(type="attention", mixer=m, mlp=f) for m, f in layers])
     if softcap is not None:

@@ -83,7 +83,7 @@ def test_residual_step(width, dtype):
         assert np.abs(h - want_h).max() < tol * max(1.0, np.abs(want_h).max())
 
 
-HEADS = [(4, 2, 64, 64), (6, 2, 48, 32), (5, 5, 40, 72), (20, 1, 16, 24), (3, 1, 128, 96), (4, 2, 256, 200), (2, 2, 12, 20), (34, 2, 8, 8), (2, 1, 300, 264)]
+HEADS = [(8, 4, 64, 64), (6, 2, 48, 32), (5, 5, 40, 72), (20, 1, 16, 24), (3, 1, 128, 96), (4, 2, 256, 200), (2, 2, 12, 20), (34, 2, 8, 8), (2, 1, 300, 264)]
 
 
 def _planted(r, T, S, H, G, dim, vdim, start, dtype):
@@ -129,7 +129,7 @@ def test_prompt_attention(H, G, dim, vdim, dtype):
     jb, r = pkg(), rng(H * 1000 + dim)
     sink = r.standard_normal(H) + 1
     tol = 3e-6 if dtype == "float32" else 1.5e-2
-    for start, T, sk, temp in ((0, 1, sink, None), (0, 2, sink, (0.5, 3)), (0, 130, sink, (0.3, 16)), (37, 65, sink, None), (63, 2, None, (0.7, 64)), (127, 200, sink, (0.5, 128))):
+    for start, T, sk, temp in ((0, 1, sink, None), (0, 2, sink, (0.5, 3)), (0, 130, sink, (0.3, 16)), (37, 65, sink, None), (63, 2, None, (0.7, 64)), (127, 200, sink, (0.4, 100))):
         q, k, v = _planted(r, T, start + T, H, G, dim, vdim, start, dtype)
         scale = 1.7 / np.sqrt(dim)
         got, want = _attend(jb, q, k, v, dtype, scale, start, sk, temp), _want(q, k, v, scale, start, sk, temp)
